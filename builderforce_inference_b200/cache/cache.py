@@ -2,7 +2,8 @@
 and per-sequence state of fixed size beside them.
 
 The model's runs say what they need (``KVNeed`` with or without a window, ``StateNeed``, or
-nothing).  Runs with the same need form a group; each group has storage, a page pool and a
+nothing).  A run that reads another run's keys and values may read them under a mask of its own;
+they are kept for whichever of the readers looks furthest.  Runs with the same need form a group; each group has storage, a page pool and a
 page table of its own, so layers that keep every key and layers that keep a window of them do
 not share pages.  A page holds ``PAGE_TOKENS`` positions as ``[kv_head][row][head_dim]``, so
 one head's rows of a page are contiguous.
@@ -17,7 +18,7 @@ token = runs * 2 * kv_heads * head_dim * element size.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Any, Dict, List, Optional, Sequence, Union
 
 import torch
@@ -42,6 +43,7 @@ class KVView:
     v_dim: Optional[int] = None        # None: as head_dim
     chunk: Optional[int] = None        # a token reads only its own block of `chunk` positions
     values_in_keys: bool = False       # a value is the first v_dim values of its key; `v` is `k`
+    keep_first: int = 0                # beside the window, a token reads the sequence's first positions
 
     @property
     def value_dim(self) -> int:
@@ -76,13 +78,23 @@ def needs_of(need) -> tuple:
     return tuple(need)
 
 
+def widened(need: KVNeed, other: KVNeed) -> KVNeed:
+    """What has to be kept so that both ``need`` and ``other`` find the positions they read."""
+    if (need.n_kv_heads, need.head_dim, need.value_dim, need.values_in_keys) != \
+            (other.n_kv_heads, other.head_dim, other.value_dim, other.values_in_keys):
+        raise CacheError(f"a run that needs {other} cannot read the cache of one that needs {need}")
+    window = None if need.window is None or other.window is None else max(need.window, other.window)
+    return replace(need, window=window, chunk=need.chunk if need.chunk == other.chunk else None,
+                   keep_first=0 if window is None else max(need.keep_first, other.keep_first))
+
+
 class _KVGroup:
     def __init__(self, need: KVNeed, keys: List[Any], n_pages: int, n_slots: int, n_blocks: int,
                  dtype: torch.dtype, device: torch.device):
         self.need = need
         self.keys = keys                       # (run, index among the run's needs) per place
         self.runs = [r for r, _ in keys]
-        self.table = PageTable(n_pages, need.window, need.chunk)
+        self.table = PageTable(n_pages, need.window, need.chunk, need.keep_first)
         self.n_blocks = n_blocks
         self.device = device
         self.storage = self.v_storage = None
@@ -122,16 +134,19 @@ class _KVGroup:
             host[:len(row)] = torch.tensor(row, dtype=torch.int32)
         self.block_dev[slot].copy_(host)
 
-    def view(self, key) -> KVView:
+    def view(self, key, mask: Optional[KVNeed] = None) -> KVView:
+        """``mask``: the need whose window, kept first positions and chunk the reader goes by (default:
+        the group's own)."""
         i = self.keys.index(key)
+        mask = self.need if mask is None else mask
         if self.need.values_in_keys:
             v = self.storage[i, 0]
         else:
             v = self.storage[i, 1] if self.v_storage is None else self.v_storage[i]
         return KVView(k=self.storage[i, 0], v=v, block_table=self.block_dev,
                       n_kv_heads=self.need.n_kv_heads, head_dim=self.need.head_dim,
-                      window=self.need.window, v_dim=self.need.v_dim, chunk=self.need.chunk,
-                      values_in_keys=self.need.values_in_keys)
+                      window=mask.window, v_dim=self.need.v_dim, chunk=mask.chunk,
+                      values_in_keys=self.need.values_in_keys, keep_first=mask.keep_first if mask.window is not None else 0)
 
     def bytes_per_token(self) -> int:
         return len(self.runs) * self.need.n_kv_heads * self.need.stored_per_head * self.storage.element_size()
@@ -200,14 +215,23 @@ class SequenceCache:
         self.state_groups: List[_StateGroup] = []
         self._owner: Dict[int, List[Any]] = {}     # run -> [(need index, group, key in the group)]
         by_need: Dict[Any, List[Any]] = {}
+        kept = {run: list(needs_of(need)) for run, need in enumerate(needs) if self.cache_of[run] is None}
+        # the masks the runs read keys and values under: the i-th of a run belongs to the i-th KVNeed it
+        # declares, which for a borrowing run stands for the i-th of the run it borrows from
+        self._masks: Dict[int, List[KVNeed]] = {}
         for run, need in enumerate(needs):
-            if self.cache_of[run] is not None:
-                src = self.cache_of[run]
-                if not 0 <= src < run or self.cache_of[src] is not None:
-                    raise CacheError(f"run {run} reads the cache of run {src}, which keeps none of its own")
+            self._masks[run] = [one for one in needs_of(need) if isinstance(one, KVNeed)]
+            src = self.cache_of[run]
+            if src is None:
                 continue
+            if not 0 <= src < run or self.cache_of[src] is not None:
+                raise CacheError(f"run {run} reads the cache of run {src}, which keeps none of its own")
+            places = [j for j, one in enumerate(kept[src]) if isinstance(one, KVNeed)]
+            for j, one in zip(places, self._masks[run]):
+                kept[src][j] = widened(kept[src][j], one)
+        for run, own in kept.items():
             self._owner[run] = []
-            for j, one in enumerate(needs_of(need)):
+            for j, one in enumerate(own):
                 # a run that names the same need twice gets two places in that need's group
                 by_need.setdefault(one, []).append((run, j))
         # parts outside the layers keep theirs under keys of their own, past the runs
@@ -236,7 +260,8 @@ class SequenceCache:
     def run_cache(self, run: int) -> RunCache:
         src = self.cache_of[run]
         owner_run = run if src is None else src
-        entries = tuple(g.view(key) if isinstance(g, _KVGroup) else g.storage[key]
+        masks = iter(self._masks[run])
+        entries = tuple(g.view(key, next(masks, None)) if isinstance(g, _KVGroup) else g.storage[key]
                         for _, g, key in self._owner.get(owner_run, ()))
         kv = next((e for e in entries if isinstance(e, KVView)), None)
         state = next((e for e in entries if not isinstance(e, KVView)), None)
@@ -363,8 +388,7 @@ class SequenceCache:
         total = 0
         for g in self.kv_groups:
             for s, n in self.lengths.items():
-                kept = n - g.table.first_kept_position(n)
-                total += kept * g.bytes_per_token()
+                total += g.table.kept_positions(n) * g.bytes_per_token()
         return total
 
     def check(self) -> None:

@@ -77,13 +77,14 @@ class PageTable:
     ``window`` and ``chunk`` are None when every earlier position is kept.  Otherwise only pages
     that still hold a position the sequence's next token may read are kept (the last ``window``
     positions; the positions of the token's own block of ``chunk`` positions); ``trim`` gives the
-    others back.
+    others back.  The pages of a sequence's first ``keep_first`` positions are never given back.
     """
 
-    def __init__(self, n_pages: int, window: Optional[int] = None, chunk: Optional[int] = None):
+    def __init__(self, n_pages: int, window: Optional[int] = None, chunk: Optional[int] = None, keep_first: int = 0):
         self.pool = FreeList(n_pages, "page")
         self.window = window
         self.chunk = chunk
+        self.keep_first = keep_first
         self.rows: Dict[int, List[int]] = {}      # slot -> page id per position block (-1: none)
 
     def open(self, slot: int) -> None:
@@ -92,13 +93,19 @@ class PageTable:
         self.rows[slot] = []
 
     def first_kept_position(self, length: int) -> int:
-        """The oldest position the next token (at ``length``) may still read."""
+        """The oldest position the next token (at ``length``) may still read, beside the first
+        ``keep_first`` ones."""
         first = 0
         if self.window is not None:
             first = max(first, length - self.window + 1)
         if self.chunk is not None:
             first = max(first, length // self.chunk * self.chunk)
         return first
+
+    def kept_positions(self, length: int) -> int:
+        """How many of a sequence's ``length`` positions the next token may still read."""
+        first = min(self.first_kept_position(length), length)
+        return length - first + min(self.keep_first, first)
 
     @property
     def keeps_everything(self) -> bool:
@@ -125,13 +132,14 @@ class PageTable:
         return changed
 
     def trim(self, slot: int, length: int) -> bool:
-        """Give back pages that lie wholly before what the token at ``length`` may read."""
+        """Give back pages that hold nothing the token at ``length``, or a later one, may read."""
         if self.keeps_everything:
             return False
         row = self.rows[slot]
         first_block = self.first_kept_position(length) // PAGE_TOKENS
         changed = False
-        for b in range(min(first_block, len(row))):
+        kept_blocks = (self.keep_first + PAGE_TOKENS - 1) // PAGE_TOKENS
+        for b in range(kept_blocks, min(first_block, len(row))):
             if row[b] >= 0:
                 self.pool.give_back(row[b])
                 row[b] = -1

@@ -6,6 +6,7 @@
 // Reference formula (crates/bfi-core/src/cpu.rs:328-392): score = q.k / sqrt(d) for keys at or
 // before the query's position, softmax over them, weighted sum of V; query head h reads kv head
 // h / (n_q / n_kv).  `window` > 0 keeps only the last `window` keys (pos - window < j <= pos).
+// `keep_first`: beside the window a query reads the first `keep_first` positions (0 <= j < keep_first).
 // `chunk` > 0 keeps only the keys of the query's own block of `chunk` consecutive positions, blocks
 // counted from position 0 of the sequence ((pos / chunk) * chunk <= j <= pos).
 // `has_sink`: the softmax's denominator carries one more term, exp(sink), a score that every
@@ -33,8 +34,8 @@ attention_paged_kernel(const T* __restrict__ q, long q_stride, T* __restrict__ o
                        const T* __restrict__ k_pages, const T* __restrict__ v_pages,
                        const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_seqlens,
                        const int* __restrict__ seq_slot, const int* __restrict__ seq_start, int n_q, int n_kv, int d,
-                       int dv, int gh, int head_chunks, int window, int chunk, float scale, int has_sink, float sink,
-                       const float* __restrict__ sinks) {
+                       int dv, int gh, int head_chunks, int window, int keep_first, int chunk, float scale, int has_sink,
+                       float sink, const float* __restrict__ sinks) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float smem[];
@@ -97,7 +98,10 @@ attention_paged_kernel(const T* __restrict__ q, long q_stride, T* __restrict__ o
     const size_t page_elems = (size_t)n_kv * BFI_PAGE_TOKENS * d;
     const size_t page_elems_v = (size_t)n_kv * BFI_PAGE_TOKENS * dv;
 
-    for (int kb = (lo / ATT_KEYS) * ATT_KEYS; kb <= hi; kb += ATT_KEYS) {
+    // the tiles of the kept first positions that lie before the window, then the window's
+    const int kb_lo = (lo / ATT_KEYS) * ATT_KEYS;
+    for (int kb = keep_first > 0 ? 0 : kb_lo; kb <= hi; kb += ATT_KEYS) {
+        if (kb >= keep_first && kb < kb_lo) kb = kb_lo;
         __syncthreads();
         const int page = block_table[(size_t)slot * table_stride + kb / BFI_PAGE_TOKENS];
         const size_t base = (size_t)(page < 0 ? 0 : page) * page_elems +
@@ -108,7 +112,7 @@ attention_paged_kernel(const T* __restrict__ q, long q_stride, T* __restrict__ o
             const int j = i / d, e = i - j * d;
             const int key = kb + j;
             float kv = 0.0f;
-            if (page >= 0 && key >= lo && key <= hi) kv = to_f32(k_pages[base + (size_t)j * d + e]);
+            if (page >= 0 && (key >= lo || key < keep_first) && key <= hi) kv = to_f32(k_pages[base + (size_t)j * d + e]);
             ks[j * (d + 1) + e] = kv;
         }
         if (v_pages != nullptr) {
@@ -116,7 +120,7 @@ attention_paged_kernel(const T* __restrict__ q, long q_stride, T* __restrict__ o
                 const int j = i / dv, e = i - j * dv;
                 const int key = kb + j;
                 float vv = 0.0f;
-                if (page >= 0 && key >= lo && key <= hi) vv = to_f32(v_pages[base_v + (size_t)j * dv + e]);
+                if (page >= 0 && (key >= lo || key < keep_first) && key <= hi) vv = to_f32(v_pages[base_v + (size_t)j * dv + e]);
                 vs[j * dv + e] = vv;
             }
         }
@@ -134,7 +138,7 @@ attention_paged_kernel(const T* __restrict__ q, long q_stride, T* __restrict__ o
         }
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-            const bool valid = row_ok[i] && page >= 0 && key <= row_pos[i] && key >= row_lo[i];
+            const bool valid = row_ok[i] && page >= 0 && key <= row_pos[i] && (key >= row_lo[i] || key < keep_first);
             const float sc = valid ? s[i] : -INFINITY;
             const float m_tile = warp_max(sc);
             if (m_tile == -INFINITY) continue;   // no key of this tile is visible to the row (uniform in the warp)
@@ -181,7 +185,7 @@ template <typename T, int NC>
 static int launch_attention(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                             const void* v_pages, const int* block_table, int table_stride, const int* cu_seqlens,
                             const int* seq_slot, const int* seq_start, int n_seqs, int max_tokens, int n_q, int n_kv,
-                            int d, int dv, int window, int chunk, float scale, int has_sink, float sink,
+                            int d, int dv, int window, int keep_first, int chunk, float scale, int has_sink, float sink,
                             const float* sinks, cudaStream_t stream) {
     const int group = n_q / n_kv;
     int gh = 1;
@@ -200,7 +204,7 @@ static int launch_attention(const void* q, long q_stride, void* out, long out_st
     }
     bfi_launch(kernel, dim3(grid), dim3(ATT_WARPS * 32), smem, stream, (const T*)q, q_stride, (T*)out, out_stride, (const T*)k_pages,
                                                    (const T*)v_pages, block_table, table_stride, cu_seqlens, seq_slot,
-                                                   seq_start, n_q, n_kv, d, dv, gh, head_chunks, window, chunk, scale, has_sink, sink, sinks);
+                                                   seq_start, n_q, n_kv, d, dv, gh, head_chunks, window, keep_first, chunk, scale, has_sink, sink, sinks);
     return bfi_check_launch("attention_paged");
 }
 
@@ -208,13 +212,13 @@ template <typename T>
 static int dispatch_nc(int nc, const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                        const void* v_pages, const int* block_table, int table_stride, const int* cu_seqlens,
                        const int* seq_slot, const int* seq_start, int n_seqs, int max_tokens, int n_q, int n_kv, int d,
-                       int dv, int window, int chunk, float scale, int has_sink, float sink, const float* sinks,
-                       cudaStream_t stream) {
+                       int dv, int window, int keep_first, int chunk, float scale, int has_sink, float sink,
+                       const float* sinks, cudaStream_t stream) {
 #define BFI_ATT_CASE(N)                                                                                              \
     case N:                                                                                                          \
         return launch_attention<T, N>(q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride,     \
                                       cu_seqlens, seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, \
-                                      chunk, scale, has_sink, sink, sinks, stream);
+                                      keep_first, chunk, scale, has_sink, sink, sinks, stream);
     switch (nc) {
         BFI_ATT_CASE(1)
         BFI_ATT_CASE(2)
@@ -233,7 +237,7 @@ static int dispatch_nc(int nc, const void* q, long q_stride, void* out, long out
 extern "C" int bfi_attention_paged(const void* q, int dtype, long q_stride, void* out, long out_stride,
                                    const void* k_pages, const void* v_pages, const int* block_table, int table_stride,
                                    const int* cu_seqlens, const int* seq_slot, const int* seq_start, int n_seqs,
-                                   int max_tokens, int n_q, int n_kv, int d, int dv, int window, int chunk, float scale,
+                                   int max_tokens, int n_q, int n_kv, int d, int dv, int window, int keep_first, int chunk, float scale,
                                    int has_sink, float sink, const float* sinks, cudaStream_t stream) {
     BFI_REQUIRE(dtype_ok(dtype), "attention_paged: unknown dtype code %d", dtype);
     BFI_REQUIRE(n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_paged: %d query heads do not divide into %d kv heads",
@@ -242,7 +246,8 @@ extern "C" int bfi_attention_paged(const void* q, int dtype, long q_stride, void
                 d, ATT_MAX_D);
     BFI_REQUIRE(dv > 0 && dv <= ATT_MAX_DV, "attention_paged: value size %d must be positive, at most %d", dv, ATT_MAX_DV);
     BFI_REQUIRE(v_pages != nullptr || dv <= d, "attention_paged: values that are the keys' first %d values need keys that long", dv);
-    BFI_REQUIRE(window >= 0 && chunk >= 0, "attention_paged: negative window or chunk");
+    BFI_REQUIRE(window >= 0 && chunk >= 0 && keep_first >= 0, "attention_paged: negative window, chunk or count of kept positions");
+    BFI_REQUIRE(keep_first == 0 || (window > 0 && chunk == 0), "attention_paged: first positions are kept beside a window");
     BFI_REQUIRE(has_sink != 2 || sinks != nullptr, "attention_paged: a sink per head needs its array");
     BFI_REQUIRE(q_stride >= (long)n_q * d && out_stride >= (long)n_q * dv, "attention_paged: token stride shorter than the heads");
     if (n_seqs <= 0 || max_tokens <= 0) return 0;
@@ -253,7 +258,7 @@ extern "C" int bfi_attention_paged(const void* q, int dtype, long q_stride, void
     if (nc > 8) nc = 16;
     if (dtype == BFI_F32)
         return dispatch_nc<float>(nc, q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride,
-                                  cu_seqlens, seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, chunk, scale, has_sink, sink, sinks, stream);
+                                  cu_seqlens, seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, keep_first, chunk, scale, has_sink, sink, sinks, stream);
     return dispatch_nc<bf16>(nc, q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride, cu_seqlens,
-                             seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, chunk, scale, has_sink, sink, sinks, stream);
+                             seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, keep_first, chunk, scale, has_sink, sink, sinks, stream);
 }

@@ -180,6 +180,9 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
 //     g' * sigmoid(alpha * g') * (u' + shift)
 // alpha 1, no limit and shift 0 is SiLU(gate) * up, and evaluates to the same bits as that formula.
 // Kind 1, the tanh form of GELU:  0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) * u.
+// With `in_scale` (float32, rows of `in_stride`) gate and up of row m and output column j are first
+// multiplied by in_scale[m][j / in_cols]: a factor per row and group of columns on the product's input
+// (an expert's weight, with the experts' columns side by side; a factor of 0 leaves 0 behind).
 // A library holds ONE set of constants per host thread (bfi_set_gate), which every product launched
 // from that thread with the gated epilogue takes along as a kernel argument.
 #define BFI_GATE_SIGMOID 0
@@ -187,8 +190,22 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
 struct GateAct {
     float alpha, limit, shift;
     int kind;
+    const float* in_scale;
+    long in_stride;
+    int in_cols;
 };
 extern thread_local GateAct g_bfi_gate;
+
+__device__ __forceinline__ float gate_in_scale(const GateAct& a, int m, int j) {
+    return a.in_scale[(size_t)m * a.in_stride + j / a.in_cols];
+}
+
+// The squared ReLU of a product that stores max(acc, 0)^2 (epilogue code 3 of the matrix products).
+#define BFI_EPI_RELU_SQUARED 3
+__device__ __forceinline__ float relu_squared(float v) {
+    v = fmaxf(v, 0.0f);
+    return v * v;
+}
 
 // 0.5 g (1 + tanh(y)) = g * sigmoid(2 y): one exponential, no cancellation for large |y|
 __device__ __forceinline__ float gelu_tanh_exact(float g) {

@@ -32,7 +32,7 @@ extern "C" int bfi_set_pdl(int on) {
 }
 
 // The constants of the gated epilogue for the products this host thread launches from now on.
-thread_local GateAct g_bfi_gate = {1.0f, 0.0f, 0.0f, BFI_GATE_SIGMOID};
+thread_local GateAct g_bfi_gate = {1.0f, 0.0f, 0.0f, BFI_GATE_SIGMOID, nullptr, 0, 1};
 
 extern "C" int bfi_set_gate(float alpha, float limit, float shift) {
     g_bfi_gate.alpha = alpha, g_bfi_gate.limit = limit, g_bfi_gate.shift = shift;
@@ -45,6 +45,13 @@ extern "C" int bfi_set_gate_kind(int kind, float alpha, float limit, float shift
     if (kind != BFI_GATE_SIGMOID && kind != BFI_GATE_GELU_TANH) return bfi_fail("set_gate_kind: unknown activation kind %d", kind);
     g_bfi_gate.alpha = alpha, g_bfi_gate.limit = limit, g_bfi_gate.shift = shift;
     g_bfi_gate.kind = kind;
+    return 0;
+}
+
+// The factors on the gated products' inputs (null: none), for the products launched from now on.
+extern "C" int bfi_set_gate_in_scale(const float* scale, long stride, int cols) {
+    if (scale != nullptr && (cols < 1 || stride < 1)) return bfi_fail("set_gate_in_scale: bad sizes cols=%d stride=%ld", cols, stride);
+    g_bfi_gate.in_scale = scale, g_bfi_gate.in_stride = stride, g_bfi_gate.in_cols = cols;
     return 0;
 }
 

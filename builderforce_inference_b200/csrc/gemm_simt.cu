@@ -9,6 +9,7 @@
 //   0  C = acc                         (C in c_dtype)
 //   1  C += acc                        (C float32: the residual stream)
 //   2  C[m, j] = silu(acc[m,2j]) * acc[m,2j+1]   (W rows interleaved gate/up; C has N/2 columns)
+//   3  C = max(acc, 0)^2               (C in c_dtype)
 #include "common.cuh"
 
 #define EPI_STORE 0
@@ -94,8 +95,10 @@ gemm_tile_kernel(const TA* __restrict__ A, long lda, const TW* __restrict__ W, l
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int gn = n0 + tx * 4 + j;
-                if (gn + 1 < N)
-                    store_from_f32(C, c_dtype, (size_t)gm * ldc + (gn >> 1), gate_mul_exact(acc[i][j], acc[i][j + 1], gate));
+                if (gn + 1 < N) {
+                    const float f = gate.in_scale ? gate_in_scale(gate, gm, gn >> 1) : 1.0f;
+                    store_from_f32(C, c_dtype, (size_t)gm * ldc + (gn >> 1), gate_mul_exact(f * acc[i][j], f * acc[i][j + 1], gate));
+                }
             }
         } else {
 #pragma unroll
@@ -106,7 +109,7 @@ gemm_tile_kernel(const TA* __restrict__ A, long lda, const TW* __restrict__ W, l
                 if (epilogue == EPI_ACCUMULATE)
                     reinterpret_cast<float*>(C)[idx] += acc[i][j];
                 else
-                    store_from_f32(C, c_dtype, idx, acc[i][j]);
+                    store_from_f32(C, c_dtype, idx, epilogue == BFI_EPI_RELU_SQUARED ? relu_squared(acc[i][j]) : acc[i][j]);
             }
         }
     }
@@ -155,13 +158,15 @@ gemv_rows_kernel(const TA* __restrict__ A, long lda, const TW* __restrict__ W, l
             const int gm = m_base + m;
             if (gm >= M) continue;
             if (epilogue == EPI_SWIGLU) {
-                if (has_b) store_from_f32(C, c_dtype, (size_t)gm * ldc + (n_a >> 1), gate_mul_exact(acc_a[m], acc_b[m], gate));
+                const float f = gate.in_scale ? gate_in_scale(gate, gm, n_a >> 1) : 1.0f;
+                if (has_b) store_from_f32(C, c_dtype, (size_t)gm * ldc + (n_a >> 1), gate_mul_exact(f * acc_a[m], f * acc_b[m], gate));
             } else if (epilogue == EPI_ACCUMULATE) {
                 reinterpret_cast<float*>(C)[(size_t)gm * ldc + n_a] += acc_a[m];
                 if (has_b) reinterpret_cast<float*>(C)[(size_t)gm * ldc + n_b] += acc_b[m];
             } else {
-                store_from_f32(C, c_dtype, (size_t)gm * ldc + n_a, acc_a[m]);
-                if (has_b) store_from_f32(C, c_dtype, (size_t)gm * ldc + n_b, acc_b[m]);
+                const bool sq = epilogue == BFI_EPI_RELU_SQUARED;
+                store_from_f32(C, c_dtype, (size_t)gm * ldc + n_a, sq ? relu_squared(acc_a[m]) : acc_a[m]);
+                if (has_b) store_from_f32(C, c_dtype, (size_t)gm * ldc + n_b, sq ? relu_squared(acc_b[m]) : acc_b[m]);
             }
         }
     }
@@ -203,7 +208,7 @@ extern "C" int bfi_gemm_simt(const void* A, int a_dtype, long lda, const void* W
     BFI_REQUIRE(dtype_ok(a_dtype) && dtype_ok(w_dtype) && dtype_ok(c_dtype), "gemm_simt: unknown dtype code");
     BFI_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm_simt: bad sizes M=%d N=%d K=%d", M, N, K);
     BFI_REQUIRE(lda >= K && ldw >= K, "gemm_simt: a row stride is shorter than K=%d", K);
-    BFI_REQUIRE(epilogue >= 0 && epilogue <= 2, "gemm_simt: unknown epilogue %d", epilogue);
+    BFI_REQUIRE(epilogue >= 0 && epilogue <= 3, "gemm_simt: unknown epilogue %d", epilogue);
     if (epilogue == EPI_ACCUMULATE) BFI_REQUIRE(c_dtype == BFI_F32, "gemm_simt: accumulation needs a float32 output");
     if (epilogue == EPI_SWIGLU) {
         BFI_REQUIRE(N % 2 == 0, "gemm_simt: the gated epilogue needs an even N, got %d", N);
@@ -214,6 +219,7 @@ extern "C" int bfi_gemm_simt(const void* A, int a_dtype, long lda, const void* W
     if (M == 0) return 0;
     // chunk M so that gridDim.y stays legal
     const int max_rows = 65535 * TM;
+    BFI_REQUIRE(M <= max_rows || g_bfi_gate.in_scale == nullptr, "gemm_simt: %d rows with input factors are too many for one launch", M);
     for (int m0 = 0; m0 < M; m0 += max_rows) {
         const int rows = M - m0 < max_rows ? M - m0 : max_rows;
         const char* a = (const char*)A + (size_t)m0 * lda * dtype_size(a_dtype);

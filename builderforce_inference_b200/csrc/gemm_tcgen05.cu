@@ -208,6 +208,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                 float v[16];
                 tmem_ld16(lane_addr + c * 16, v);
                 if (epilogue == EPI_SWIGLU) {
+                    if (gate.in_scale != nullptr) {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j)
+                            v[j] *= (j < rows_here && n < N) ? gate_in_scale(gate, m_c + j, n >> 1) : 0.0f;
+                    }
 #pragma unroll
                     for (int j = 0; j < 16; ++j) v[j] = gate_mul_fast(v[j], __shfl_down_sync(0xffffffffu, v[j], 1), gate);
                     if ((lane & 1) == 0 && n + 1 < N) {
@@ -225,6 +230,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         for (int j = 0; j < 16; ++j)
                             if (j < rows_here) c_io[(size_t)j * ldc] = old[j] + v[j];
                     } else {
+                        if (epilogue == BFI_EPI_RELU_SQUARED) {
+#pragma unroll
+                            for (int j = 0; j < 16; ++j) v[j] = relu_squared(v[j]);
+                        }
 #pragma unroll
                         for (int j = 0; j < 16; ++j)
                             if (j < rows_here) store_from_f32(C, c_dtype, (size_t)(m_c + j) * ldc + n, v[j]);
@@ -282,6 +291,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                     for (int r = 0; r < 8; ++r) v += x[u][r];
                     if (epilogue == EPI_SWIGLU) {
+                        if (gate.in_scale != nullptr) v *= (live && n < N) ? gate_in_scale(gate, m, n >> 1) : 0.0f;
                         const float act = gate_mul_fast(v, __shfl_down_sync(0xffffffffu, v, 1), gate);
                         if (live && (lane & 1) == 0 && n + 1 < N) store_from_f32(C, c_dtype, (size_t)m * ldc + (n >> 1), act);
                     } else if (live && n < N) {
@@ -289,7 +299,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         if (epilogue == EPI_ACCUMULATE)
                             reinterpret_cast<float*>(C)[o] = old[u] + v;
                         else
-                            store_from_f32(C, c_dtype, o, v);
+                            store_from_f32(C, c_dtype, o, epilogue == BFI_EPI_RELU_SQUARED ? relu_squared(v) : v);
                     }
                 }
             }
@@ -438,6 +448,28 @@ __device__ __forceinline__ void tp_emit_group(uint4* stage, const float (&v)[G][
     }
 }
 
+
+// What happens to 16 accumulators (features n .. n+15 of token m) before they are stored: the squared
+// ReLU, or the factors on the gated product's input.  in_cols is a multiple of 8 in most models: the
+// chunk's 8 output columns then share one factor.
+__device__ __forceinline__ void tp_pre_store(float (&v)[16], int epilogue, const GateAct& gate, int m, int n, int M, int N) {
+    if (epilogue == BFI_EPI_RELU_SQUARED) {
+#pragma unroll
+        for (int j = 0; j < 16; ++j) v[j] = relu_squared(v[j]);
+    } else if (epilogue == EPI_SWIGLU && gate.in_scale != nullptr) {
+        if ((gate.in_cols & 7) == 0) {
+            const float f = (m < M && n < N) ? gate_in_scale(gate, m, n >> 1) : 0.0f;
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] *= f;
+        } else {
+#pragma unroll
+            for (int j = 0; j < 16; j += 2) {
+                const float f = (m < M && n + j < N) ? gate_in_scale(gate, m, (n + j) >> 1) : 0.0f;
+                v[j] *= f, v[j + 1] *= f;
+            }
+        }
+    }
+}
 
 template <int HALVES>
 __global__ void __launch_bounds__(TP_THREADS, 1)
@@ -635,11 +667,15 @@ gemm_tcgen05_prefill_kernel(const __grid_constant__ CUtensorMap map_a, const __g
                     if (!wide && c_direct + 4 <= c_end && n0 + 64 <= N) {
                         float v[4][16];
                         tmem_ld64(taddr + c_direct * 16, v);
+#pragma unroll
+                        for (int g = 0; g < 4; ++g) tp_pre_store(v[g], epilogue, gate, m, n0 + g * 16, M, N);
                         tp_emit_group<4>(stage, v, lane, epilogue, gate, c_dtype, C, ldc, m_base, M, n0);
                         c_direct += 4;
                     } else if (c_direct + 2 <= c_end && n0 + 32 <= N) {
                         float v[2][16];
                         tmem_ld32(taddr + c_direct * 16, v);
+#pragma unroll
+                        for (int g = 0; g < 2; ++g) tp_pre_store(v[g], epilogue, gate, m, n0 + g * 16, M, N);
                         tp_emit_group<2>(stage, v, lane, epilogue, gate, c_dtype, C, ldc, m_base, M, n0);
                         c_direct += 2;
                     } else {
@@ -654,6 +690,7 @@ gemm_tcgen05_prefill_kernel(const __grid_constant__ CUtensorMap map_a, const __g
                 float v[16];
                 tmem_ld16(taddr + c * 16, v);
                 if (m >= M) continue;
+                tp_pre_store(v, epilogue, gate, m, n, M, N);
                 const bool whole = vec_ok && n + 16 <= N;
                 if (epilogue == EPI_SWIGLU) {
                     if (whole) {
@@ -965,7 +1002,7 @@ static int gemm_tcgen05_launch(const void* A, long lda, const void* W, long ldw,
                                int N, int K, int epilogue, int* status, cudaStream_t stream, TcWaits waits) {
     BFI_REQUIRE(dtype_ok(c_dtype), "gemm_tcgen05: unknown output dtype code %d", c_dtype);
     BFI_REQUIRE(M >= 0 && N > 0 && K > 0, "gemm_tcgen05: bad sizes M=%d N=%d K=%d", M, N, K);
-    BFI_REQUIRE(epilogue >= 0 && epilogue <= 2, "gemm_tcgen05: unknown epilogue %d", epilogue);
+    BFI_REQUIRE(epilogue >= 0 && epilogue <= 3, "gemm_tcgen05: unknown epilogue %d", epilogue);
     BFI_REQUIRE(status != nullptr, "gemm_tcgen05: a status word is required");
     if (epilogue == EPI_ACCUMULATE) BFI_REQUIRE(c_dtype == BFI_F32, "gemm_tcgen05: accumulation needs a float32 output");
     if (epilogue == EPI_SWIGLU) BFI_REQUIRE(N % 2 == 0, "gemm_tcgen05: the gated epilogue needs an even N, got %d", N);

@@ -9,12 +9,14 @@
 // `vb` columns of one head of one sequence and walks the sequence's new tokens in order.  Thread
 // (g, c) of a block holds rows g, g + groups, ... of column c in shared memory.
 //
+// q and k may be rotated (value i with value i + dims/2 of a head's first `dims` values, by the angle
+// of the token's position) and k multiplied by a constant, in float32 as they are read (LightRot).
+//
 // After the recurrence the heads of a token are normalised together and gated:
 //     y = o * rsqrt(mean(o^2) + eps) * w * sigmoid(gate)        (bfi_gated_rmsnorm)
 #include "common.cuh"
 
-#define LIGHT_ACT_NONE 0
-#define LIGHT_ACT_SILU 1
+#include "lightning.cuh"
 
 __device__ __forceinline__ float light_silu(float x) {
     float s;
@@ -32,12 +34,39 @@ __device__ __forceinline__ float light_sigmoid(float x) {
     return z / (1.0f + z);
 }
 
+// q and k of one head of the token at row `row` (its q and k heads at qh and kh), activated, rotated and
+// scaled, into shared memory.
+template <typename T>
+__device__ __forceinline__ void light_load_qk(const T* __restrict__ qh, const T* __restrict__ kh, float* qs, float* ks, int D,
+                                              int act, const LightRot& rot, int pos) {
+    const bool turn = rot.table != nullptr && light_position_ok(rot, pos);
+    const int half = rot.dims >> 1;
+    const float2* cs = turn ? rot.table + (size_t)pos * half : nullptr;
+    auto value = [&](const T* p, int j) {
+        const float x = to_f32(p[j]);
+        return act == LIGHT_ACT_SILU ? light_silu(x) : x;
+    };
+    for (int j = threadIdx.x; j < D; j += blockDim.x) {
+        float qv = value(qh, j), kv = value(kh, j);
+        if (turn && j < rot.dims) {
+            const bool first = j < half;
+            const int other = first ? j + half : j - half;
+            const float2 c = cs[first ? j : other];
+            const float qo = value(qh, other), ko = value(kh, other);
+            qv = first ? qv * c.x - qo * c.y : qv * c.x + qo * c.y;
+            kv = first ? kv * c.x - ko * c.y : kv * c.x + ko * c.y;
+        }
+        qs[j] = qv;
+        ks[j] = kv * rot.k_scale;
+    }
+}
+
 template <typename T>
 __global__ void lightning_scan_kernel(const T* __restrict__ proj, long stride, int q_off, int k_off, int v_off,
                                       float* __restrict__ out, long out_stride, float* __restrict__ state,
                                       const float* __restrict__ decay, const int* __restrict__ cu_seqlens,
                                       const int* __restrict__ seq_slot, int H, int D, int V, int vb, int v_blocks,
-                                      int act) {
+                                      int act, const LightRot rot) {
     pdl_trigger();
     extern __shared__ float sm[];
     float* S = sm;                     // [D][vb]
@@ -59,11 +88,7 @@ __global__ void lightning_scan_kernel(const T* __restrict__ proj, long stride, i
     pdl_wait();
     for (int t = 0; t < nt; ++t) {
         const T* row = proj + (size_t)(t0 + t) * stride + (size_t)h * D;
-        for (int j = threadIdx.x; j < D; j += blockDim.x) {
-            const float qv = to_f32(row[q_off + j]), kv = to_f32(row[k_off + j]);
-            qs[j] = act == LIGHT_ACT_SILU ? light_silu(qv) : qv;
-            ks[j] = act == LIGHT_ACT_SILU ? light_silu(kv) : kv;
-        }
+        light_load_qk(row + q_off, row + k_off, qs, ks, D, act, rot, rot.table ? rot.token_pos[t0 + t] : 0);
         float vv = 0.0f;
         if (col_ok) {
             vv = to_f32(proj[(size_t)(t0 + t) * stride + v_off + (size_t)h * V + v0 + c]);
@@ -100,7 +125,7 @@ __global__ void __launch_bounds__(LIGHT_STEP_COLS * LIGHT_STEP_GROUPS)
 lightning_step_kernel(const T* __restrict__ proj, long stride, int q_off, int k_off, int v_off, float* __restrict__ out,
                       long out_stride, float* __restrict__ state, const float* __restrict__ decay,
                       const int* __restrict__ cu_seqlens, const int* __restrict__ seq_slot, int H, int D, int V,
-                      int v_blocks, int act) {
+                      int v_blocks, int act, const LightRot rot) {
     pdl_trigger();
     __shared__ float qs[LIGHT_STEP_GROUPS * RPT], ks[LIGHT_STEP_GROUPS * RPT];
     __shared__ float red[LIGHT_STEP_GROUPS][LIGHT_STEP_COLS];
@@ -122,11 +147,7 @@ lightning_step_kernel(const T* __restrict__ proj, long stride, int q_off, int k_
     pdl_wait();
     const int t = cu_seqlens[seq];
     const T* row = proj + (size_t)t * stride;
-    for (int j = threadIdx.x; j < D; j += blockDim.x) {
-        const float qv = to_f32(row[q_off + (size_t)h * D + j]), kv = to_f32(row[k_off + (size_t)h * D + j]);
-        qs[j] = act == LIGHT_ACT_SILU ? light_silu(qv) : qv;
-        ks[j] = act == LIGHT_ACT_SILU ? light_silu(kv) : kv;
-    }
+    light_load_qk(row + q_off + (size_t)h * D, row + k_off + (size_t)h * D, qs, ks, D, act, rot, rot.table ? rot.token_pos[t] : 0);
     float vv = 0.0f;
     if (col_ok) {
         vv = to_f32(row[v_off + (size_t)h * V + v0 + c]);
@@ -156,12 +177,12 @@ lightning_step_kernel(const T* __restrict__ proj, long stride, int q_off, int k_
 template <typename T>
 static bool launch_light_step(const void* proj, long stride, int q_off, int k_off, int v_off, float* out, long out_stride,
                               float* state, const float* decay, const int* cu_seqlens, const int* seq_slot, int n_seqs,
-                              int H, int D, int V, int act, cudaStream_t stream) {
+                              int H, int D, int V, int act, const LightRot& rot, cudaStream_t stream) {
     const int v_blocks = (V + LIGHT_STEP_COLS - 1) / LIGHT_STEP_COLS;
     const dim3 grid(H * v_blocks, n_seqs), block(LIGHT_STEP_COLS * LIGHT_STEP_GROUPS);
 #define BFI_LIGHT_STEP(R)                                                                                              \
     bfi_launch(lightning_step_kernel<T, R>, grid, block, 0, stream, (const T*)proj, stride, q_off, k_off, v_off, out,  \
-               out_stride, state, decay, cu_seqlens, seq_slot, H, D, V, v_blocks, act)
+               out_stride, state, decay, cu_seqlens, seq_slot, H, D, V, v_blocks, act, rot)
     if (D <= 32) BFI_LIGHT_STEP(4);
     else if (D <= 64) BFI_LIGHT_STEP(8);
     else if (D <= 128) BFI_LIGHT_STEP(16);
@@ -174,7 +195,11 @@ static bool launch_light_step(const void* proj, long stride, int q_off, int k_of
 extern "C" int bfi_lightning_scan(const void* proj, int dtype, long stride, int q_off, int k_off, int v_off, float* out,
                                   long out_stride, float* state, const float* decay, const int* cu_seqlens,
                                   const int* seq_slot, int n_seqs, int H, int D, int V, int act, int few_tokens,
-                                  cudaStream_t stream) {
+                                  const void* rope_table, int rot_dims, int table_positions, const int* token_pos, float k_scale,
+                                  int* status, cudaStream_t stream) {
+    const LightRot rot = {(const float2*)rope_table, rot_dims, table_positions, token_pos, k_scale, status};
+    BFI_REQUIRE(rope_table == nullptr || (rot_dims > 0 && rot_dims % 2 == 0 && rot_dims <= D && table_positions > 0 && token_pos != nullptr),
+                "lightning_scan: a rotation of %d of %d values needs an even width, a table and the tokens' positions", rot_dims, D);
     BFI_REQUIRE(dtype_ok(dtype), "lightning_scan: unknown dtype code %d", dtype);
     BFI_REQUIRE(H > 0 && D > 0 && V > 0, "lightning_scan: bad sizes heads=%d dim=%d vdim=%d", H, D, V);
     BFI_REQUIRE(act == LIGHT_ACT_NONE || act == LIGHT_ACT_SILU, "lightning_scan: unknown activation %d", act);
@@ -182,8 +207,8 @@ extern "C" int bfi_lightning_scan(const void* proj, int dtype, long stride, int 
     if (n_seqs <= 0) return 0;
     if (few_tokens == 2 && n_seqs <= 65535) {      // every sequence brings exactly one token: the state stays in registers
         const bool ran = dtype == BFI_F32
-            ? launch_light_step<float>(proj, stride, q_off, k_off, v_off, out, out_stride, state, decay, cu_seqlens, seq_slot, n_seqs, H, D, V, act, stream)
-            : launch_light_step<bf16>(proj, stride, q_off, k_off, v_off, out, out_stride, state, decay, cu_seqlens, seq_slot, n_seqs, H, D, V, act, stream);
+            ? launch_light_step<float>(proj, stride, q_off, k_off, v_off, out, out_stride, state, decay, cu_seqlens, seq_slot, n_seqs, H, D, V, act, rot, stream)
+            : launch_light_step<bf16>(proj, stride, q_off, k_off, v_off, out, out_stride, state, decay, cu_seqlens, seq_slot, n_seqs, H, D, V, act, rot, stream);
         if (ran) return bfi_check_launch("lightning_step");
     }
     // columns per block: few where the step is short (more blocks share the state's traffic)
@@ -202,12 +227,12 @@ extern "C" int bfi_lightning_scan(const void* proj, int dtype, long stride, int 
         if (smem > 48 * 1024) e = cudaFuncSetAttribute(lightning_scan_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess)
             bfi_launch(lightning_scan_kernel<float>, dim3(H * v_blocks, n_seqs), dim3(threads), smem, stream, (const float*)proj,
-                       stride, q_off, k_off, v_off, out, out_stride, state, decay, cu_seqlens, seq_slot, H, D, V, vb, v_blocks, act);
+                       stride, q_off, k_off, v_off, out, out_stride, state, decay, cu_seqlens, seq_slot, H, D, V, vb, v_blocks, act, rot);
     } else {
         if (smem > 48 * 1024) e = cudaFuncSetAttribute(lightning_scan_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess)
             bfi_launch(lightning_scan_kernel<bf16>, dim3(H * v_blocks, n_seqs), dim3(threads), smem, stream, (const bf16*)proj,
-                       stride, q_off, k_off, v_off, out, out_stride, state, decay, cu_seqlens, seq_slot, H, D, V, vb, v_blocks, act);
+                       stride, q_off, k_off, v_off, out, out_stride, state, decay, cu_seqlens, seq_slot, H, D, V, vb, v_blocks, act, rot);
     }
     if (e != cudaSuccess) return bfi_fail("lightning_scan: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     return bfi_check_launch("lightning_scan");

@@ -13,11 +13,15 @@
 //     `score_mode` 1: s = sigmoid(z), every expert by itself, instead of the softmax.
 //     `group_top` g > 1: a group's score is the sum of its g largest choice scores (of all of them,
 //     if it has fewer) instead of the largest.
-// `act_kind` of the experts: 0 = silu(gate) * up over interleaved gate and up rows (W_gu as below);
+//     `dense_weight` (float32 [tokens, E], optional) receives every expert's weight, 0 where it was not
+//     chosen (and in padding rows): the factors of a dense product that computes all experts.
+// `act_kind` of the experts: 0 = the gated activation of common.cuh with its slope, clamp and shift (silu(gate)
+//     * up by default) over interleaved gate and up rows (W_gu as below); `in_weight` (float32 per pair) multiplies
+//     the expert's input, and so its gate and up;
 //     1 = relu(up)^2, no gate: W_gu is then [E * ff, width], expert e's up row j at row e ff + j.
 // bfi_moe_router: the same decision with the logits made here, z = W_router h (float32 rows of W).
 // bfi_moe_gate_up:  act[t, k, :] = silu(W_gate[e] h_t) * (W_up[e] h_t),  e = idx[t, k]
-// bfi_moe_down:     out[t, :] (= | +=) sum_k weight[t, k] * W_down[idx[t, k]] act[t, k, :]
+// bfi_moe_down:     out[t, :] (= | +=) sum_k weight[t, k] * W_down[idx[t, k]] act[t, k, :]     (no weights: 1)
 //                                      + gate[t] * shared[t, :]            (the last term optional)
 // The experts' weights are two matrices for all experts, the layouts the dense products take as well:
 // W_gu [E * 2 * ff, width], expert e's gate row j at row 2 (e ff + j) and its up row right after it;
@@ -40,7 +44,10 @@ __device__ __forceinline__ float moe_sigmoid(float x) {
 __device__ __forceinline__ void moe_route_token(const float* zr, const float* __restrict__ correction, int* __restrict__ idx,
                                                 float* __restrict__ weight, float* __restrict__ gate, float* s, float* choice,
                                                 float* gs, int t, int E, int top, int n_groups, int keep, float weight_scale,
-                                                int extra, int lane, int score_mode, int group_top) {
+                                                int extra, int lane, int score_mode, int group_top,
+                                                float* __restrict__ dense_weight) {
+    if (dense_weight != nullptr)
+        for (int e = lane; e < E; e += 32) dense_weight[(size_t)t * E + e] = 0.0f;
     if (score_mode == 1) {
         for (int e = lane; e < E; e += 32) {
             s[e] = moe_sigmoid(zr[e]);
@@ -127,7 +134,9 @@ __device__ __forceinline__ void moe_route_token(const float* zr, const float* __
         if (at == 0x7fffffff) at = 0;                  // nothing left to choose from: expert 0 with weight 0
         if (lane == 0) {
             idx[(size_t)t * top + r] = at;
-            weight[(size_t)t * top + r] = best == -INFINITY ? 0.0f : s[at] * weight_scale;
+            const float w = best == -INFINITY ? 0.0f : s[at] * weight_scale;
+            weight[(size_t)t * top + r] = w;
+            if (dense_weight != nullptr && best != -INFINITY) dense_weight[(size_t)t * E + at] = w;
             choice[at] = NAN;                          // taken
         }
         __syncwarp();
@@ -148,7 +157,7 @@ __global__ void moe_route_kernel(const float* __restrict__ z, long z_stride, con
     if (t >= n_tokens) return;
     float* s = sm + (size_t)warp * (2 * E + n_groups);
     moe_route_token(z + (size_t)t * z_stride, correction, idx, weight, gate, s, s + E, s + 2 * E, t, E, top, n_groups, keep,
-                    weight_scale, extra, lane, score_mode, group_top);
+                    weight_scale, extra, lane, score_mode, group_top, nullptr);
 }
 
 extern "C" int bfi_moe_route(const float* z, long z_stride, const float* correction, int* idx, float* weight, float* gate,
@@ -221,14 +230,19 @@ __global__ void __launch_bounds__(256)
 moe_router_kernel(const T* __restrict__ h, long h_stride, const float* __restrict__ w_router,
                   const float* __restrict__ correction, const int* __restrict__ token_slot, int* __restrict__ idx,
                   float* __restrict__ weight, float* __restrict__ gate, int width, int E, int top, int n_groups, int keep,
-                  float weight_scale, int extra, int score_mode, int group_top) {
+                  float weight_scale, int extra, int score_mode, int group_top, float* __restrict__ dense_weight) {
     pdl_trigger();
     extern __shared__ __align__(16) float sm[];
     float* hs = sm;                                // [width]
     float* z = hs + width;                         // [E + 1]
     float* scratch = z + E + 1;                    // [2 E + n_groups]
     const int t = blockIdx.x;
-    if (token_slot[t] < 0) return;
+    if (token_slot[t] < 0) {                       // padding row
+        pdl_wait();
+        if (dense_weight != nullptr)
+            for (int e = threadIdx.x; e < E; e += blockDim.x) dense_weight[(size_t)t * E + e] = 0.0f;
+        return;
+    }
     pdl_wait();
     for (int j = threadIdx.x; j < width; j += blockDim.x) hs[j] = to_f32(h[(size_t)t * h_stride + j]);
     __syncthreads();
@@ -240,13 +254,13 @@ moe_router_kernel(const T* __restrict__ h, long h_stride, const float* __restric
     __syncthreads();
     if (warp == 0)
         moe_route_token(z, correction, idx, weight, gate, scratch, scratch + E, scratch + 2 * E, t, E, top, n_groups, keep,
-                        weight_scale, extra, lane, score_mode, group_top);
+                        weight_scale, extra, lane, score_mode, group_top, dense_weight);
 }
 
 extern "C" int bfi_moe_router(const void* h, long h_stride, int dtype, const float* w_router, const float* correction,
                               const int* token_slot, int* idx, float* weight, float* gate, int n_tokens, int width, int E,
                               int top, int n_groups, int keep, float weight_scale, int extra, int score_mode, int group_top,
-                              cudaStream_t stream) {
+                              float* dense_weight, cudaStream_t stream) {
     BFI_REQUIRE(dtype_ok(dtype), "moe_router: unknown dtype code %d", dtype);
     BFI_REQUIRE((score_mode == 0 || score_mode == 1) && group_top >= 1, "moe_router: unknown score mode or group rule");
     BFI_REQUIRE(E > 0 && top > 0 && top <= E && width > 0 && h_stride >= width, "moe_router: cannot choose %d of %d experts", top, E);
@@ -262,12 +276,14 @@ extern "C" int bfi_moe_router(const void* h, long h_stride, int dtype, const flo
         if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_router_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess)
             bfi_launch(moe_router_kernel<float>, dim3(n_tokens), dim3(256), smem, stream, (const float*)h, h_stride, w_router, correction,
-                       token_slot, idx, weight, gate, width, E, top, n_groups, keep, weight_scale, extra, score_mode, group_top);
+                       token_slot, idx, weight, gate, width, E, top, n_groups, keep, weight_scale, extra, score_mode, group_top,
+                       dense_weight);
     } else {
         if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_router_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess)
             bfi_launch(moe_router_kernel<bf16>, dim3(n_tokens), dim3(256), smem, stream, (const bf16*)h, h_stride, w_router, correction,
-                       token_slot, idx, weight, gate, width, E, top, n_groups, keep, weight_scale, extra, score_mode, group_top);
+                       token_slot, idx, weight, gate, width, E, top, n_groups, keep, weight_scale, extra, score_mode, group_top,
+                       dense_weight);
     }
     if (e != cudaSuccess) return bfi_fail("moe_router: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     return bfi_check_launch("moe_router");
@@ -280,7 +296,7 @@ template <typename T>
 __global__ void __launch_bounds__(MOE_WARPS * 32)
 moe_gate_up_kernel(const T* __restrict__ h, long h_stride, const T* __restrict__ w_gu,
                    const int* __restrict__ idx, const int* __restrict__ token_slot, T* __restrict__ act, int top,
-                   int width, int ff, int rows_per_block, int act_kind) {
+                   int width, int ff, int rows_per_block, int act_kind, const GateAct gate, const float* __restrict__ in_weight) {
     pdl_trigger();
     extern __shared__ __align__(16) float hs[];    // [width]
     const int pair = blockIdx.x;
@@ -300,17 +316,21 @@ moe_gate_up_kernel(const T* __restrict__ h, long h_stride, const T* __restrict__
         }
         return;
     }
+    const float f = in_weight != nullptr ? in_weight[pair] : 1.0f;
     for (int r = r0 + warp; r < r1; r += MOE_WARPS) {
         const size_t off = ((size_t)e * ff + r) * 2 * width;
         const float g = warp_dot<T>(w_gu + off, hs, width, lane);
         const float u = warp_dot<T>(w_gu + off + width, hs, width, lane);
-        if (lane == 0) act[(size_t)pair * ff + r] = from_f32<T>(g * moe_sigmoid(g) * u);
+        if (lane == 0) act[(size_t)pair * ff + r] = from_f32<T>(gate_mul_exact(f * g, f * u, gate));
     }
 }
 
 extern "C" int bfi_moe_gate_up(const void* h, long h_stride, int dtype, const void* w_gu,
                                const int* idx, const int* token_slot, void* act, int n_tokens, int top, int width, int ff,
-                               int act_kind, cudaStream_t stream) {
+                               int act_kind, float gate_alpha, float gate_limit, float gate_shift, const float* in_weight,
+                               cudaStream_t stream) {
+    const GateAct gate = {gate_alpha, gate_limit, gate_shift, BFI_GATE_SIGMOID, nullptr, 0, 1};
+    BFI_REQUIRE(act_kind == 0 || in_weight == nullptr, "moe_gate_up: an input weight needs gated experts");
     BFI_REQUIRE(dtype_ok(dtype), "moe_gate_up: unknown dtype code %d", dtype);
     BFI_REQUIRE(act_kind == 0 || act_kind == 1, "moe_gate_up: unknown activation kind %d", act_kind);
     BFI_REQUIRE(top > 0 && width > 0 && ff > 0 && h_stride >= width, "moe_gate_up: bad sizes");
@@ -331,12 +351,12 @@ extern "C" int bfi_moe_gate_up(const void* h, long h_stride, int dtype, const vo
         if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_gate_up_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess)
             bfi_launch(moe_gate_up_kernel<float>, grid, dim3(MOE_WARPS * 32), smem, stream, (const float*)h, h_stride,
-                       (const float*)w_gu, idx, token_slot, (float*)act, top, width, ff, rows_per_block, act_kind);
+                       (const float*)w_gu, idx, token_slot, (float*)act, top, width, ff, rows_per_block, act_kind, gate, in_weight);
     } else {
         if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_gate_up_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e == cudaSuccess)
             bfi_launch(moe_gate_up_kernel<bf16>, grid, dim3(MOE_WARPS * 32), smem, stream, (const bf16*)h, h_stride,
-                       (const bf16*)w_gu, idx, token_slot, (bf16*)act, top, width, ff, rows_per_block, act_kind);
+                       (const bf16*)w_gu, idx, token_slot, (bf16*)act, top, width, ff, rows_per_block, act_kind, gate, in_weight);
     }
     if (e != cudaSuccess) return bfi_fail("moe_gate_up: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
     return bfi_check_launch("moe_gate_up");
@@ -365,7 +385,7 @@ moe_down_kernel(const T* __restrict__ act, const T* __restrict__ w_down, const i
         for (int k = 0; k < top; ++k) {
             const int e = idx[(size_t)t * top + k];
             const float d = warp_dot<T>(w_down + (size_t)c * ld + (size_t)e * ff, as + (size_t)k * ff, ff, lane);
-            sum = fmaf(weight[(size_t)t * top + k], d, sum);
+            sum = fmaf(weight != nullptr ? weight[(size_t)t * top + k] : 1.0f, d, sum);
         }
         if (lane == 0) {
             if (shared_out) sum = fmaf(g, shared_out[(size_t)t * shared_stride + c], sum);

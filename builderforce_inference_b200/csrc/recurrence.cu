@@ -946,7 +946,7 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ x, long x_stri
         for (int j = lane; j < len; j += 32) {
             const float gv = to_f32(gr[j0 + j]);
             const float ga = gate_act ? rec_silu(gv) : rec_sigmoid(gv);
-            yr[j0 + j] = from_f32<T>(xr[j0 + j] * ga * scale * load_as_f32(w, w_dtype, (j0 + j) % w_len));
+            yr[j0 + j] = from_f32<T>(xr[j0 + j] * ga * scale * (w != nullptr ? load_as_f32(w, w_dtype, (j0 + j) % w_len) : 1.0f));
         }
     }
 }

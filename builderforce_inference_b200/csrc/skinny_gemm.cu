@@ -217,7 +217,8 @@ __global__ void skinny_gemm_kernel(const bf16* __restrict__ A, long lda, const b
             const int m = idx / PAIRS, p = idx - m * PAIRS;
             const int row = row0 + 2 * p;
             if (m >= M || row + 1 >= N) continue;
-            store_from_f32(C, c_dtype, (size_t)m * ldc + (row >> 1), gate_mul_fast(total(2 * p, m), total(2 * p + 1, m), gate));
+            const float f = gate.in_scale ? gate_in_scale(gate, m, row >> 1) : 1.0f;
+            store_from_f32(C, c_dtype, (size_t)m * ldc + (row >> 1), gate_mul_fast(f * total(2 * p, m), f * total(2 * p + 1, m), gate));
         }
     } else {
         for (int idx = threadIdx.x; idx < R * MP; idx += blockDim.x) {
@@ -229,7 +230,7 @@ __global__ void skinny_gemm_kernel(const bf16* __restrict__ A, long lda, const b
             if (epilogue == EPI_ACCUMULATE)
                 reinterpret_cast<float*>(C)[o] += v;
             else
-                store_from_f32(C, c_dtype, o, v);
+                store_from_f32(C, c_dtype, o, epilogue == BFI_EPI_RELU_SQUARED ? relu_squared(v) : v);
         }
     }
 }
@@ -326,7 +327,7 @@ static int skinny_check_args(const void* A, long lda, const void* W, long ldw, i
                              int epilogue) {
     BFI_REQUIRE(dtype_ok(c_dtype), "skinny_gemm: unknown output dtype code %d", c_dtype);
     BFI_REQUIRE(M >= 0 && N > 0 && K > 0, "skinny_gemm: bad sizes M=%d N=%d K=%d", M, N, K);
-    BFI_REQUIRE(epilogue >= 0 && epilogue <= 2, "skinny_gemm: unknown epilogue %d", epilogue);
+    BFI_REQUIRE(epilogue >= 0 && epilogue <= 3, "skinny_gemm: unknown epilogue %d", epilogue);
     if (epilogue == EPI_ACCUMULATE) BFI_REQUIRE(c_dtype == BFI_F32, "skinny_gemm: accumulation needs a float32 output");
     if (epilogue == EPI_SWIGLU) BFI_REQUIRE(N % 2 == 0, "skinny_gemm: the gated epilogue needs an even N, got %d", N);
     if (M == 0) return 0;

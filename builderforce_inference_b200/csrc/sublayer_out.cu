@@ -9,6 +9,7 @@
 //                      h[t, :] = x[t, :] * rsqrt(mean(x[t, :]^2) + eps2) * w2       (h in the activation dtype)
 //   bfi_weighted_sum:  out[t, :] = a * y0[t, :] + b * y1[t, :]                      (all float32)
 //   bfi_scale_rows:    x[r, :] *= s                                                 (float32)
+//   bfi_softcap_rows:  x[r, :] = cap * tanh(x[r, :] / cap)                          (float32)
 //   bfi_gated_rows:    out[r, :] (= | +=) g[r] * src[r, :]                          (float32)
 //
 // The residual stream x and the sublayer outputs are float32 in every run dtype; the weight is
@@ -336,6 +337,25 @@ extern "C" int bfi_scale_rows(float* x, long stride, int n_rows, int cols, float
     BFI_REQUIRE(n_rows <= 65535, "scale_rows: %d rows are too many for one launch", n_rows);
     bfi_launch(scale_rows_kernel, dim3((cols + 255) / 256, n_rows), dim3(256), 0, stream, x, stride, cols, s);
     return bfi_check_launch("scale_rows");
+}
+
+__global__ void softcap_rows_kernel(float* __restrict__ x, long stride, int cols, float cap) {
+    pdl_trigger();
+    pdl_wait();
+    float* r = x + (size_t)blockIdx.y * stride;
+    const int j = blockIdx.x * blockDim.x + threadIdx.x;
+    if (j < cols) r[j] = cap * tanhf(r[j] / cap);
+}
+
+// x[r, :] = cap * tanh(x[r, :] / cap) over float32 rows (soft-capped logits)
+extern "C" int bfi_softcap_rows(float* x, long stride, int n_rows, int cols, float cap, cudaStream_t stream) {
+    BFI_REQUIRE(n_rows >= 0 && cols > 0 && stride >= cols, "softcap_rows: bad sizes rows=%d cols=%d", n_rows, cols);
+    BFI_REQUIRE(cap > 0.0f, "softcap_rows: the cap must be positive");
+    for (int r0 = 0; r0 < n_rows; r0 += 65535) {
+        const int rows = n_rows - r0 < 65535 ? n_rows - r0 : 65535;
+        bfi_launch(softcap_rows_kernel, dim3((cols + 255) / 256, rows), dim3(256), 0, stream, x + (size_t)r0 * stride, stride, cols, cap);
+    }
+    return bfi_check_launch("softcap_rows");
 }
 
 __global__ void gated_rows_kernel(float* __restrict__ out, long out_stride, const float* __restrict__ src, long src_stride,

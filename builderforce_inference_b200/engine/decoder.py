@@ -165,6 +165,7 @@ class Decoder:
             ctx.extras["next_run"] = cache.run_cache(i + 1) if follows else None
             self.blocks[self.spec.schedule[i].layer].forward(ctx, x, cache.run_cache(i))
         ctx.extras.pop("outnorm.input", None)
+        ctx.extras.pop("sandwich.input", None)
 
     def logits(self, ctx, x: torch.Tensor, rows: torch.Tensor, out: torch.Tensor) -> None:
         """Final norm and head at the given rows of ``x``; ``out`` is float32 ``[len(rows), vocab]``."""
@@ -172,3 +173,5 @@ class Decoder:
         linear(h, self.head, out, EPI_STORE)
         if self.spec.logit_scale != 1.0:
             ops.scale_rows(out, float(self.spec.logit_scale))
+        if self.spec.logit_softcap is not None:
+            ops.softcap_rows(out, float(self.spec.logit_softcap))

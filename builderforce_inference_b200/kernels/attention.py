@@ -8,7 +8,7 @@ import torch
 def attend(ctx, qkv, out, kv, n_heads: int, scale: float, sink=None, exact_weights: bool = False) -> bool:
     """``exact_weights``: the design wants its attention weights in float32; only kernels that keep
     them so (in effect) are chosen."""
-    if qkv.dtype != torch.bfloat16:
+    if qkv.dtype != torch.bfloat16 or kv.keep_first:
         return False
     if not kv.plain or isinstance(sink, torch.Tensor) or exact_weights:
         # a chunked mask or a learned sink per head: steps with more than one token per sequence have

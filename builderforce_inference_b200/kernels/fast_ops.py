@@ -8,7 +8,7 @@ from ctypes import c_float, c_int, c_long
 import torch
 
 from .library import KernelError, library
-from .ops import _ptr, _rows_2d, _stream, dtype_code
+from .ops import LIGHT_ACT_SILU, _ptr, _rows_2d, _stream, dtype_code, rotation_args
 
 SKINNY_MAX_ROWS = 64
 
@@ -338,17 +338,20 @@ LIGHTNING_CHUNK_MIN_TOKENS = 8     # shorter runs of new tokens: the token-by-to
 
 def lightning_chunks_bf16(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, out: torch.Tensor, state: torch.Tensor,
                           decay: torch.Tensor, cu_seqlens: torch.Tensor, seq_slot: torch.Tensor, n_seqs: int,
-                          n_heads: int, dim: int, vdim: int) -> bool:
+                          n_heads: int, dim: int, vdim: int, act: int = LIGHT_ACT_SILU, rope_table=None, rot_dim: int = 0,
+                          token_pos=None, k_scale: float = 1.0, status=None) -> bool:
     """The decayed linear attention over runs of new tokens, 64 at a time on the tensor cores (SiLU
-    on q, k, v applied as they are read).  Same arguments and state as ``ops.lightning_scan``;
-    False for sizes it does not take (head sizes that are no multiples of 16, or too large)."""
+    on q, k, v, or their rotation and scale, applied as they are read).  Same arguments and state as
+    ``ops.lightning_scan``; False for sizes it does not take (head sizes that are no multiples of 16, or
+    too large; a rotation whose halves are no multiples of 8)."""
     if proj.dtype != torch.bfloat16 or out.dtype != torch.float32 or state.dtype != torch.float32:
         return False
     _rows_2d(proj, "projections")
     _rows_2d(out, "recurrence output")
     if not state.is_contiguous() or tuple(state.shape[1:]) != (n_heads, dim, vdim) or out.shape[1] != n_heads * vdim:
         raise KernelError("lightning_chunks: state [slots, heads, dim, vdim] and output [tokens, heads * vdim] expected")
+    rope = rotation_args(rope_table, rot_dim, token_pos, proj.shape[0])
     return library("fast").call_optional(
         "bfi_lightning_chunks_bf16", _ptr(proj), c_long(proj.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off),
         _ptr(out), c_long(out.stride(0)), _ptr(state), _ptr(decay), _ptr(cu_seqlens), _ptr(seq_slot), c_int(n_seqs),
-        c_int(n_heads), c_int(dim), c_int(vdim), _stream())
+        c_int(n_heads), c_int(dim), c_int(vdim), c_int(act), *rope, c_float(k_scale), _ptr(status), _stream())

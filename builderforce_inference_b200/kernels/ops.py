@@ -15,6 +15,7 @@ from .library import KernelError, library
 EPI_STORE = 0
 EPI_ACCUMULATE = 1
 EPI_SWIGLU = 2
+EPI_RELU_SQUARED = 3
 
 FLAG_WRITE_CACHE = 1
 FLAG_K_IN_PLACE = 2
@@ -257,16 +258,34 @@ def qk_prepare(qkv: torch.Tensor, n_q: int, n_kv: int, head_dim: int, token_pos:
 LIGHT_ACT_NONE, LIGHT_ACT_SILU = 0, 1
 
 
+def rotation_args(table: Optional[torch.Tensor], rot_dim: int, token_pos: Optional[torch.Tensor], n_tokens: int) -> list:
+    """A rotation table (float32 ``[positions, rot_dim/2, 2]``, or None), its width, its positions and
+    the tokens' positions, checked, as launch arguments."""
+    if table is None:
+        return [_ptr(None), c_int(0), c_int(0), _ptr(None)]
+    if table.dtype != torch.float32 or not table.is_contiguous() or table.dim() != 3 or table.shape[1] != rot_dim // 2 \
+            or table.shape[2] != 2:
+        raise KernelError("rotation table must be contiguous float32 [positions, rot_dim/2, 2]")
+    if token_pos is None or token_pos.numel() < n_tokens:
+        raise KernelError("a rotation needs the position of every token")
+    _i32(token_pos, "token positions")
+    return [_ptr(table), c_int(rot_dim), c_int(table.shape[0]), _ptr(token_pos)]
+
+
 def lightning_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, out: torch.Tensor, state: torch.Tensor,
                    decay: torch.Tensor, cu_seqlens: torch.Tensor, seq_slot: torch.Tensor, n_seqs: int,
                    n_heads: int, dim: int, vdim: int, act: int = LIGHT_ACT_SILU, few_tokens: bool = False,
-                   single_tokens: bool = False) -> None:
+                   single_tokens: bool = False, rope_table: Optional[torch.Tensor] = None, rot_dim: int = 0,
+                   token_pos: Optional[torch.Tensor] = None, k_scale: float = 1.0,
+                   status: Optional[torch.Tensor] = None) -> None:
     """Linear attention with a decay per head over the step's new tokens, sequence by sequence:
     ``S = decay * S + k v^T; o = S^T q`` with ``S`` float32 ``[slots, heads, dim, vdim]`` carried
     in ``state``.  q, k, v are columns ``q_off``, ``k_off``, ``v_off`` of ``proj`` (activated here
     when ``act`` says so); ``out`` is float32 ``[tokens, heads * vdim]``.  ``single_tokens``: every
-    sequence of the step brings exactly one token (the kernel then keeps the state in registers)."""
-    _need_cuda(proj, out, state, decay, cu_seqlens, seq_slot)
+    sequence of the step brings exactly one token (the kernel then keeps the state in registers).
+    With ``rope_table`` the first ``rot_dim`` values of every q and k head are rotated (value i with value
+    i + rot_dim/2) by the token's position, and k is multiplied by ``k_scale``, both in float32."""
+    _need_cuda(proj, out, state, decay, cu_seqlens, seq_slot, rope_table, token_pos, status)
     _rows_2d(proj, "projections")
     _rows_2d(out, "recurrence output")
     _i32(cu_seqlens, "cu_seqlens")
@@ -279,10 +298,12 @@ def lightning_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, out: 
         raise KernelError("lightning_scan: one float32 decay per head")
     if max(q_off, k_off) + n_heads * dim > proj.shape[1] or v_off + n_heads * vdim > proj.shape[1]:
         raise KernelError("lightning_scan: the projections' row is shorter than the heads")
+    rope = rotation_args(rope_table, rot_dim, token_pos, proj.shape[0])
     library("core").call("bfi_lightning_scan", _ptr(proj), c_int(dtype_code(proj.dtype)), c_long(proj.stride(0)),
                          c_int(q_off), c_int(k_off), c_int(v_off), _ptr(out), c_long(out.stride(0)), _ptr(state),
                          _ptr(decay), _ptr(cu_seqlens), _ptr(seq_slot), c_int(n_seqs), c_int(n_heads), c_int(dim),
-                         c_int(vdim), c_int(act), c_int(2 if single_tokens else (1 if few_tokens else 0)), _stream())
+                         c_int(vdim), c_int(act), c_int(2 if single_tokens else (1 if few_tokens else 0)), *rope,
+                         c_float(k_scale), _ptr(status), _stream())
 
 
 def gated_rmsnorm(x: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor) -> None:
@@ -330,8 +351,8 @@ def attention_paged(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv, cu_se
         c_long(out.stride(0)), _ptr(kv.k), _ptr(None if kv.values_in_keys else kv.v), _ptr(kv.block_table),
         c_int(kv.block_table.stride(0)),
         _ptr(cu_seqlens), _ptr(seq_slot), _ptr(seq_start), c_int(n_seqs), c_int(max_tokens), c_int(n_q),
-        c_int(kv.n_kv_heads), c_int(kv.head_dim), c_int(kv.value_dim), c_int(kv.window or 0), c_int(kv.chunk or 0),
-        c_float(scale), c_int(has_sink), c_float(sink_value), _ptr(sinks), _stream())
+        c_int(kv.n_kv_heads), c_int(kv.head_dim), c_int(kv.value_dim), c_int(kv.window or 0), c_int(kv.keep_first),
+        c_int(kv.chunk or 0), c_float(scale), c_int(has_sink), c_float(sink_value), _ptr(sinks), _stream())
 
 
 def latent_prepare(proj: torch.Tensor, qa: torch.Tensor, n_heads: int, dim: int, rot_dim: int, rank: int, kv_off: int,
@@ -536,6 +557,16 @@ def scale_rows(x: torch.Tensor, s: float) -> None:
                          c_float(s), _stream())
 
 
+def softcap_rows(x: torch.Tensor, cap: float) -> None:
+    """``x = cap * tanh(x / cap)`` over float32 rows."""
+    _need_cuda(x)
+    _rows_2d(x, "rows")
+    if x.dtype != torch.float32 or not cap > 0.0:
+        raise KernelError("softcap_rows: float32 rows and a positive cap")
+    library("core").call("bfi_softcap_rows", _ptr(x), c_long(x.stride(0)), c_int(x.shape[0]), c_int(x.shape[1]),
+                         c_float(cap), _stream())
+
+
 def gated_rows(out: torch.Tensor, src: torch.Tensor, g: torch.Tensor, accumulate: bool = False) -> None:
     """``out[r] (= | +=) g[r] * src[r]`` over float32 rows, one factor per row."""
     _need_cuda(out, src, g)
@@ -732,10 +763,10 @@ def sigmoid_gate(x: torch.Tensor, g: torch.Tensor, group: int) -> None:
 GATE_SIGMOID, GATE_SILU = 0, 1
 
 
-def gated_group_norm(x: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor, parts: int,
+def gated_group_norm(x: torch.Tensor, gate: torch.Tensor, w: Optional[torch.Tensor], eps: float, out: torch.Tensor, parts: int,
                      gate_first: bool, gate_act: int = GATE_SILU) -> None:
     """A row cut into ``parts`` equal parts, each divided by its own root mean square, times ``w``
-    (which repeats along the row when shorter), with a gate ``act(gate)`` applied before the norm
+    (which repeats along the row when shorter; None: no weight), with a gate ``act(gate)`` applied before the norm
     (``gate_first``) or after it.  ``x`` float32; ``gate`` and ``out`` in the activation dtype."""
     _need_cuda(x, gate, w, out)
     _rows_2d(x, "norm input")
@@ -744,16 +775,17 @@ def gated_group_norm(x: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: 
     n, width = x.shape
     if x.dtype != torch.float32 or gate.dtype != out.dtype or gate.shape != (n, width) or out.shape != (n, width):
         raise KernelError("gated_group_norm: x float32 [rows, width]; gate and output [rows, width] of one dtype")
-    if w.dim() != 1 or not w.is_contiguous():
+    if w is not None and (w.dim() != 1 or not w.is_contiguous()):
         raise KernelError("gated_group_norm: the weight must be a contiguous vector")
     library("core").call("bfi_gated_group_norm", _ptr(x), c_long(x.stride(0)), _ptr(gate), c_long(gate.stride(0)),
-                         c_int(dtype_code(out.dtype)), _ptr(w), c_int(dtype_code(w.dtype)), c_int(w.numel()), _ptr(out),
+                         c_int(dtype_code(out.dtype)), _ptr(w), c_int(0 if w is None else dtype_code(w.dtype)),
+                         c_int(1 if w is None else w.numel()), _ptr(out),
                          c_long(out.stride(0)), c_int(n), c_int(width), c_int(parts), c_int(1 if gate_first else 0),
                          c_int(gate_act), c_float(eps), _stream())
 
 
 SCORE_SOFTMAX, SCORE_SIGMOID = 0, 1
-EXPERT_GATED_SILU, EXPERT_RELU_SQUARED = 0, 1
+EXPERT_GATED, EXPERT_RELU_SQUARED = 0, 1
 
 
 def moe_route(z: torch.Tensor, n_experts: int, correction: Optional[torch.Tensor], idx: torch.Tensor,
@@ -784,10 +816,14 @@ def moe_route(z: torch.Tensor, n_experts: int, correction: Optional[torch.Tensor
 def moe_router(h: torch.Tensor, w_router: torch.Tensor, n_experts: int, correction: Optional[torch.Tensor],
                token_slot: torch.Tensor, idx: torch.Tensor, weight: torch.Tensor, top: int, n_groups: int = 1, keep: int = 1,
                weight_scale: float = 1.0, gate: Optional[torch.Tensor] = None, score: int = SCORE_SOFTMAX,
-               group_top: int = 1) -> None:
+               group_top: int = 1, dense_weight: Optional[torch.Tensor] = None) -> None:
     """``moe_route`` with the logits made in the same kernel: ``z = w_router h`` with ``w_router``
-    float32 ``[n_experts (+ 1), width]`` (the extra row is the gate's, wanted with ``gate``)."""
-    _need_cuda(h, w_router, correction, token_slot, idx, weight, gate)
+    float32 ``[n_experts (+ 1), width]`` (the extra row is the gate's, wanted with ``gate``).
+    ``dense_weight`` (float32 ``[tokens, n_experts]``) receives every expert's weight, 0 for those not chosen."""
+    _need_cuda(h, w_router, correction, token_slot, idx, weight, gate, dense_weight)
+    if dense_weight is not None and (dense_weight.dtype != torch.float32 or not dense_weight.is_contiguous()
+                                     or dense_weight.shape != (h.shape[0], n_experts)):
+        raise KernelError("moe_router: the dense weights must be contiguous float32 [tokens, experts]")
     _rows_2d(h, "router input")
     n, width = h.shape
     rows = n_experts + (0 if gate is None else 1)
@@ -803,12 +839,15 @@ def moe_router(h: torch.Tensor, w_router: torch.Tensor, n_experts: int, correcti
     library("core").call("bfi_moe_router", _ptr(h), c_long(h.stride(0)), c_int(dtype_code(h.dtype)), _ptr(w_router),
                          _ptr(correction), _ptr(token_slot), _ptr(idx), _ptr(weight), _ptr(gate), c_int(n), c_int(width),
                          c_int(n_experts), c_int(top), c_int(n_groups), c_int(keep), c_float(weight_scale),
-                         c_int(0 if gate is None else 1), c_int(score), c_int(group_top), _stream())
+                         c_int(0 if gate is None else 1), c_int(score), c_int(group_top), _ptr(dense_weight), _stream())
 
 
 def moe_gate_up(h: torch.Tensor, w_gu: torch.Tensor, n_experts: int, idx: torch.Tensor, token_slot: torch.Tensor,
-                act: torch.Tensor, kind: int = EXPERT_GATED_SILU) -> None:
-    """``act[t, k] = silu(gate_e h_t) * (up_e h_t)`` with ``e = idx[t, k]``; ``w_gu`` is
+                act: torch.Tensor, kind: int = EXPERT_GATED, gate_act=(1.0, 0.0, 0.0),
+                in_weight: Optional[torch.Tensor] = None) -> None:
+    """``act[t, k] = silu(gate_e h_t) * (up_e h_t)`` (or another member of the gated family: ``gate_act`` is
+    its slope, clamp and shift, see ``gate_mul``; ``in_weight`` float32 ``[tokens, top]`` multiplies the
+    expert's input) with ``e = idx[t, k]``; ``w_gu`` is
     ``[experts * 2 * ff, width]`` with expert e's gate row j at row ``2 (e ff + j)`` and its up row
     after it, ``act`` ``[tokens * top, ff]``.  ``EXPERT_RELU_SQUARED``: ``act[t, k] = relu(up_e h_t)^2``
     with ``w_gu`` ``[experts * ff, width]``, the experts' up matrices one after the other.  ``idx``
@@ -827,16 +866,17 @@ def moe_gate_up(h: torch.Tensor, w_gu: torch.Tensor, n_experts: int, idx: torch.
         raise KernelError("moe_gate_up: the output must be contiguous [tokens * top, ff] of the input's dtype")
     _i32(idx, "expert choices")
     _i32(token_slot, "token slots")
+    _f32_vector(in_weight, n * top, "moe_gate_up: the input weights")
     library("core").call("bfi_moe_gate_up", _ptr(h), c_long(h.stride(0)), c_int(dtype_code(h.dtype)), _ptr(w_gu),
                          _ptr(idx), _ptr(token_slot), _ptr(act), c_int(n), c_int(top), c_int(width), c_int(ff), c_int(kind),
-                         _stream())
+                         c_float(gate_act[0]), c_float(gate_act[1]), c_float(gate_act[2]), _ptr(in_weight), _stream())
 
 
-def moe_down(act: torch.Tensor, w_down: torch.Tensor, n_experts: int, idx: torch.Tensor, weight: torch.Tensor,
+def moe_down(act: torch.Tensor, w_down: torch.Tensor, n_experts: int, idx: torch.Tensor, weight: Optional[torch.Tensor],
              token_slot: torch.Tensor, out: torch.Tensor, shared_out: Optional[torch.Tensor] = None,
              gate: Optional[torch.Tensor] = None, accumulate: bool = False) -> None:
     """``out[t] (= | +=) sum_k weight[t, k] * down_e act[t, k] + gate[t] * shared_out[t]`` with
-    ``e = idx[t, k]`` (the last term only with ``shared_out``; ``gate`` None is 1); ``w_down`` is
+    ``e = idx[t, k]`` (the last term only with ``shared_out``; ``weight`` and ``gate`` None are 1); ``w_down`` is
     ``[width, experts * ff]`` with expert e's columns at ``e ff`` (its rows may be further apart: the
     first columns of a wider matrix), ``out`` float32 ``[tokens, width]``."""
     _need_cuda(act, w_down, idx, weight, token_slot, out, shared_out, gate)
@@ -860,7 +900,7 @@ def moe_down(act: torch.Tensor, w_down: torch.Tensor, n_experts: int, idx: torch
 
 def moe_weigh_dense(act: torch.Tensor, n_experts: int, idx: torch.Tensor, weight: torch.Tensor,
                     token_slot: torch.Tensor, tail: int = 0, gate: Optional[torch.Tensor] = None,
-                    kind: int = EXPERT_GATED_SILU) -> None:
+                    kind: int = EXPERT_GATED) -> None:
     """``act[t, e ff + j] *= (weight of expert e for token t, 0 if it was not chosen)`` over
     activations ``[tokens, experts * ff + tail]`` that the dense product computed for every expert;
     the last ``tail`` columns (an expert every token uses) are multiplied by ``gate[t]`` (None: 1).
@@ -875,7 +915,7 @@ def moe_weigh_dense(act: torch.Tensor, n_experts: int, idx: torch.Tensor, weight
     if act.shape[0] != n or tail < 0 or routed <= 0 or routed % n_experts != 0 or weight.dtype != torch.float32 \
             or not weight.is_contiguous() or weight.shape != (n, top):
         raise KernelError("moe_weigh_dense: activations [tokens, experts * ff + tail], weights float32 [tokens, top]")
-    if tail and kind == EXPERT_GATED_SILU and gate is None:
+    if tail and kind == EXPERT_GATED and gate is None:
         raise KernelError("moe_weigh_dense: the tail needs one float32 gate per token")
     if gate is not None and (gate.dtype != torch.float32 or not gate.is_contiguous() or gate.numel() < n):
         raise KernelError("moe_weigh_dense: the gate must be contiguous float32 with one value per token")

@@ -18,6 +18,7 @@ rotation); ``sink`` (a score every query sees beside its keys, with no value: th
 denominator carries ``exp(sink)``; a number, or ``"learned"``: one per query head, a tensor of the
 checkpoint); ``v_dim`` (value heads of another size than the keys'); ``chunk`` (a token reads only
 the keys of its own block of ``chunk`` consecutive positions, blocks counted from position 0);
+``keep_first`` (beside its window a token reads the sequence's first ``keep_first`` positions);
 ``out_bias`` (whether the output projection carries a bias when the others do; default: it does);
 ``exact_weights`` (the softmax's weights stay float32 up to the second product, also in a bfloat16
 run: the tensor-core prompt kernel then multiplies with two bfloat16 terms per weight);
@@ -55,7 +56,8 @@ class Attention(Mixer):
                  window: Optional[int] = None, scale: Optional[float] = None, own_kv: bool = True,
                  bias: bool = False, values: str = "projection", sink=None, v_dim: Optional[int] = None,
                  chunk: Optional[int] = None, out_bias: Optional[bool] = None, exact_weights: bool = False,
-                 conv_taps: Optional[int] = None, v_mix: Optional[str] = None, gate: Optional[str] = None):
+                 conv_taps: Optional[int] = None, v_mix: Optional[str] = None, gate: Optional[str] = None,
+                 keep_first: int = 0):
         if n_heads % n_kv_heads != 0:
             raise ValueError(f"GQA: {n_heads} query heads do not divide into {n_kv_heads} kv heads")
         if head_dim % 2 != 0 or head_dim > 512:
@@ -72,6 +74,8 @@ class Attention(Mixer):
             raise ValueError(f"window must be positive, got {window}")
         if chunk is not None and chunk < 1:
             raise ValueError(f"chunk must be positive, got {chunk}")
+        if keep_first < 0 or (keep_first > 0 and chunk is not None):
+            raise ValueError(f"first positions are kept beside a window, not beside a chunk; got keep_first {keep_first}")
         v_dim = head_dim if v_dim is None else int(v_dim)
         if v_dim < 1 or v_dim > 512:
             raise ValueError(f"attention kernels take value sizes from 1 to 512, got {v_dim}")
@@ -92,6 +96,7 @@ class Attention(Mixer):
         self.taps, self.v_mix, self.gate = (None if conv_taps is None else int(conv_taps)), v_mix, gate
         self.width, self.n_heads, self.n_kv_heads, self.head_dim = width, n_heads, n_kv_heads, head_dim
         self.qk_norm, self.eps, self.window = (qk_norm or None), float(eps), window
+        self.keep_first = int(keep_first) if window is not None else 0
         self.bias, self.values_are_keys = bool(bias), values == "keys"
         self.v_dim, self.chunk, self.exact_weights = v_dim, chunk, bool(exact_weights)
         self.out_bias = self.bias if out_bias is None else bool(out_bias)
@@ -144,7 +149,7 @@ class Attention(Mixer):
 
     def cache_need(self):
         kv = KVNeed(self.n_kv_heads, self.head_dim, self.window,
-                    v_dim=None if self.v_dim == self.head_dim else self.v_dim, chunk=self.chunk)
+                    v_dim=None if self.v_dim == self.head_dim else self.v_dim, chunk=self.chunk, keep_first=self.keep_first)
         if self.taps is None or self.taps == 1:
             return kv
         return (kv, StateNeed((self.taps - 1, self._n_qkv()), "float32"))

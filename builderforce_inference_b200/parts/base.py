@@ -60,9 +60,11 @@ class ParamSpec:
 class KVNeed:
     """A mixer that keeps keys and values of earlier tokens: all of them, a window (the last
     ``window`` positions), or the current chunk (the positions of the token's own block of ``chunk``
-    consecutive positions, blocks counted from position 0).  ``v_dim`` is the size of a value head
-    where it differs from the keys' ``head_dim``.  ``values_in_keys``: a token's value is the first
-    ``v_dim`` values of its key, so only keys are stored (a latent attention's cache row)."""
+    consecutive positions, blocks counted from position 0).  Beside a window, the first
+    ``keep_first`` positions stay readable for good.  ``v_dim`` is the size of a value head where it
+    differs from the keys' ``head_dim``.  ``values_in_keys``: a token's value is the first ``v_dim``
+    values of its key, so only keys are stored (a latent attention's cache row).  A run that reads
+    another run's cache names what it reads itself; the cache keeps what any of its readers needs."""
 
     n_kv_heads: int
     head_dim: int
@@ -70,6 +72,7 @@ class KVNeed:
     v_dim: Optional[int] = None
     chunk: Optional[int] = None
     values_in_keys: bool = False
+    keep_first: int = 0
 
     @property
     def value_dim(self) -> int:
@@ -271,5 +274,6 @@ class ModelSpec:
     stop_ids: Tuple[int, ...] = ()
     embedding_scale: float = 1.0       # the embedding rows are multiplied by it; the tied head is not
     logit_scale: float = 1.0           # the logits are multiplied by it
+    logit_softcap: Optional[float] = None   # c: the logits become c * tanh(logits / c)
     # parts added to the embedded tokens, each with the checkpoint names of its tensors: (PartSpec, names)
     input_parts: Sequence[Tuple[PartSpec, Mapping[str, str]]] = ()

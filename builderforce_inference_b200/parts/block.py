@@ -9,7 +9,8 @@ the mixer's and the feed-forward's last matrix product.
               x += norm2b(ffn(norm2(x)))``; the feed-forward (with its two norms) may be absent.
               The sublayers write their output to a float32 buffer (``forward_store``) and the
               second norm adds it, normed, into the residual stream in one kernel, which also makes
-              the feed-forward's input norm.
+              the norm in front of the sublayer that follows: the feed-forward's, or that of the
+              sandwich block that runs next.
 ``outnorm``   a norm on each sublayer's OUTPUT only; the sublayers read the residual stream itself:
               ``x += mult * norm1(g1 * mixer(c1(x))); x += mult * norm2(g2 * ffn(c2(x)))``.  ``c`` is the
               identity or, with ``conv_taps``, ``c(x)_t = x_t + sum_j w[:, j] x_(t - taps + 1 + j)``, a
@@ -117,14 +118,19 @@ class SandwichBlock(Block):
     def forward(self, ctx, residual, run) -> None:
         import torch
         y = ctx.rows("sublayer.out", residual.shape[1], torch.float32)
-        h = self.norm1.forward(ctx, residual)
+        after = ctx.extras.get("next_block")
+        then = after.norm1 if isinstance(after, SandwichBlock) else None
+        made = ctx.extras.pop("sandwich.input", None)
+        h = made[1] if made is not None and made[0] is self else self.norm1.forward(ctx, residual)
         self._mixer.forward_store(ctx, h, y, run)
         if self.ffn is None:
-            self.norm1b.add_to(ctx, residual, y)
-            return
-        h = self.norm1b.add_to(ctx, residual, y, then=self.norm2)      # the add and the next norm in one kernel
-        self.ffn.forward_store(ctx, h, y)
-        self.norm2b.add_to(ctx, residual, y)
+            h = self.norm1b.add_to(ctx, residual, y, then=then)
+        else:
+            h = self.norm1b.add_to(ctx, residual, y, then=self.norm2)      # the add and the next norm in one kernel
+            self.ffn.forward_store(ctx, h, y)
+            h = self.norm2b.add_to(ctx, residual, y, then=then)
+        if then is not None:
+            ctx.extras["sandwich.input"] = (after, h)
 
 
 @BLOCKS.register("outnorm")

@@ -14,7 +14,9 @@ three constants do not apply to it.
 
 ``dense_mlp`` is the feed-forward without a gate: ``W_down act(W_up h + b_up) + b_down`` with the tanh
 GELU; the biases may be absent.  The kernel that applies bias and activation also writes ``b_down``
-into the float32 target rows, into which the down product then accumulates.
+into the float32 target rows, into which the down product then accumulates.  ``activation``
+``"relu_squared"`` (without biases) is ``W_down max(W_up h, 0)^2``, the activation applied by the up product
+as it stores.
 """
 from __future__ import annotations
 
@@ -23,7 +25,7 @@ from typing import Dict
 import torch
 
 from ..kernels import ops
-from ..kernels.linear import EPI_ACCUMULATE, EPI_STORE, EPI_SWIGLU, GATE_GELU_TANH, linear
+from ..kernels.linear import EPI_ACCUMULATE, EPI_RELU_SQUARED, EPI_STORE, EPI_SWIGLU, GATE_GELU_TANH, linear
 from .base import FEED_FORWARDS, FeedForward, ParamSpec
 
 
@@ -71,8 +73,11 @@ class DenseMLP(FeedForward):
     graph_safe = True
 
     def __init__(self, width: int, inner: int, activation: str = "gelu_tanh", bias: bool = True):
-        if activation != "gelu_tanh":
-            raise ValueError(f"dense_mlp supports the gelu_tanh activation, got {activation!r}")
+        if activation not in ("gelu_tanh", "relu_squared"):
+            raise ValueError(f"dense_mlp supports the gelu_tanh and relu_squared activations, got {activation!r}")
+        if activation == "relu_squared" and bias:
+            raise ValueError("dense_mlp: the squared ReLU takes no biases")
+        self.activation = activation
         self.width, self.inner, self.bias = int(width), int(inner), bool(bias)
         self.w_up = self.w_down = self.b_up = self.b_down = None
 
@@ -89,6 +94,10 @@ class DenseMLP(FeedForward):
 
     def forward_store(self, ctx, h, out) -> None:
         act = ctx.rows("mlp.act", self.inner)
+        if self.activation == "relu_squared":
+            linear(h, self.w_up, act, EPI_RELU_SQUARED)
+            linear(act, self.w_down, out, EPI_STORE)
+            return
         linear(h, self.w_up, act, EPI_STORE)
         if self.bias:
             ops.bias_act(act, self.b_up, act, fill=out, fill_bias=self.b_down)
@@ -98,6 +107,11 @@ class DenseMLP(FeedForward):
             linear(act, self.w_down, out, EPI_STORE)
 
     def forward(self, ctx, h, residual) -> None:
+        if self.activation == "relu_squared":
+            act = ctx.rows("mlp.act", self.inner)
+            linear(h, self.w_up, act, EPI_RELU_SQUARED)
+            linear(act, self.w_down, residual, EPI_ACCUMULATE)
+            return
         y = ctx.rows("mlp.out", self.width, torch.float32)
         self.forward_store(ctx, h, y)
         ops.residual_add(residual, y)

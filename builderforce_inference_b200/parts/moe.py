@@ -27,7 +27,13 @@ of the softmax); ``group_top`` (a group counts by the sum of its ``group_top`` b
 instead of the best one); ``correction`` false (no stored vector: experts are chosen by ``s``);
 ``expert`` ``"relu_squared"`` (an expert is ``W_down relu(W_up h)^2``, without a gate matrix: the up
 matrices of all experts are one matrix, and in the dense way the activation is applied by the
-kernel that weighs); ``shared_gate`` false (the shared expert is added as it is).
+kernel that weighs); ``shared_gate`` false (the shared expert is added as it is); ``gate_alpha``,
+``limit``, ``up_shift`` (the gated experts' activation as in ``parts/mlp.py``:
+``g' * sigmoid(gate_alpha * g') * (u' + up_shift)`` with gate and up clamped at ``limit``); ``weight_on``
+``"input"`` (the sum of ``expert(weight * h)`` instead of ``weight * expert(h)``: gate and up are linear in h,
+so both are multiplied by the weight before the activation, in float32; in the dense way the router
+kernel leaves every expert's weight, 0 for those not chosen, and the first product's epilogue multiplies by
+it, which needs no kernel between the two products).
 """
 from __future__ import annotations
 
@@ -49,7 +55,8 @@ class RoutedMLP(FeedForward):
 
     def __init__(self, width: int, n_experts: int, top: int, inner: int, n_groups: int = 1, keep_groups: int = 1,
                  shared_inner: Optional[int] = None, correction: bool = True, weight_scale: float = 1.0,
-                 score: str = "softmax", group_top: int = 1, expert: str = "gated_silu", shared_gate: bool = True):
+                 score: str = "softmax", group_top: int = 1, expert: str = "gated_silu", shared_gate: bool = True,
+                 gate_alpha: float = 1.0, limit: Optional[float] = None, up_shift: float = 0.0, weight_on: str = "output"):
         if n_experts < 1 or not 1 <= top <= n_experts or inner < 1:
             raise ValueError(f"routed feed-forward: bad sizes experts={n_experts} top={top} inner={inner}")
         if n_groups < 1 or n_experts % n_groups != 0 or not 1 <= keep_groups <= n_groups:
@@ -65,7 +72,19 @@ class RoutedMLP(FeedForward):
         self.score = ops.SCORE_SIGMOID if score == "sigmoid" else ops.SCORE_SOFTMAX
         self.group_top = int(group_top)
         self.gated = expert == "gated_silu"
-        self.kind = ops.EXPERT_GATED_SILU if self.gated else ops.EXPERT_RELU_SQUARED
+        self.kind = ops.EXPERT_GATED if self.gated else ops.EXPERT_RELU_SQUARED
+        if limit is not None and not limit > 0:
+            raise ValueError(f"routed feed-forward: the clamp limit must be positive, got {limit}")
+        self.gate_act = (float(gate_alpha), 0.0 if limit is None else float(limit), float(up_shift))
+        plain = self.gate_act == (1.0, 0.0, 0.0)
+        if not plain and (not self.gated or self.shared_inner is not None):
+            raise ValueError("routed feed-forward: slope, clamp and shift belong to gated experts without a shared one")
+        self.epilogue_gate = None if plain else self.gate_act
+        if weight_on not in ("output", "input"):
+            raise ValueError(f"routed feed-forward: weight_on must be 'output' or 'input', got {weight_on!r}")
+        self.weight_input = weight_on == "input"
+        if self.weight_input and (not self.gated or self.shared_inner is not None):
+            raise ValueError("routed feed-forward: weights on the input belong to gated experts without a shared one")
         self.shared_gate = bool(shared_gate) and self.shared_inner is not None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
@@ -131,13 +150,20 @@ class RoutedMLP(FeedForward):
         idx = ctx.rows("moe.idx", self.top, torch.int32)
         wts = ctx.rows("moe.weight", self.top, torch.float32)
         gate = ctx.rows("moe.gate", 1, torch.float32).view(-1) if self.shared_gate else None
+        dense = h.dtype == torch.bfloat16 and self.w_gu_all.dtype == torch.bfloat16 \
+            and n * self.top >= DENSE_PAIRS_PER_EXPERT * self.n_experts
+        every = ctx.rows("moe.weight.dense", self.n_experts, torch.float32) if dense and self.weight_input else None
         ops.moe_router(h, self.w_router, self.n_experts, self.correction, ctx.token_slot, idx, wts, self.top, self.n_groups,
-                       self.keep_groups, self.weight_scale, gate, self.score, self.group_top)
-        if h.dtype == torch.bfloat16 and self.w_gu_all.dtype == torch.bfloat16 \
-                and n * self.top >= DENSE_PAIRS_PER_EXPERT * self.n_experts:
+                       self.keep_groups, self.weight_scale, gate, self.score, self.group_top, dense_weight=every)
+        if dense and self.weight_input:
+            act = ctx.rows("moe.act.dense", self.n_experts * self.inner)
+            linear(h, self.w_gu_all, act, EPI_SWIGLU, self.epilogue_gate, in_scale=(every, self.inner))
+            linear(act, self.w_down_all, target, EPI_ACCUMULATE if accumulate else EPI_STORE)
+            return
+        if dense:
             tail = self.shared_inner or 0
             act = ctx.rows("moe.act.dense", self.n_experts * self.inner + tail)
-            linear(h, self.w_gu_all, act, EPI_SWIGLU if self.gated else EPI_STORE)
+            linear(h, self.w_gu_all, act, EPI_SWIGLU if self.gated else EPI_STORE, self.epilogue_gate)
             ops.moe_weigh_dense(act, self.n_experts, idx, wts, ctx.token_slot, tail, gate, self.kind)
             linear(act, self.w_down_all, target, EPI_ACCUMULATE if accumulate else EPI_STORE)
             return
@@ -151,5 +177,7 @@ class RoutedMLP(FeedForward):
             ys = ctx.rows("moe.shared.out", self.width, torch.float32)
             linear(act_s, self.ws_down, ys, EPI_STORE)
         act = ctx.rows("moe.act", self.top * self.inner).view(n * self.top, self.inner)
-        ops.moe_gate_up(h, self.w_gu, self.n_experts, idx, ctx.token_slot, act, self.kind)
-        ops.moe_down(act, self.w_down, self.n_experts, idx, wts, ctx.token_slot, target, ys, gate, accumulate)
+        ops.moe_gate_up(h, self.w_gu, self.n_experts, idx, ctx.token_slot, act, self.kind, self.gate_act,
+                        wts if self.weight_input else None)
+        ops.moe_down(act, self.w_down, self.n_experts, idx, None if self.weight_input else wts, ctx.token_slot, target, ys, gate,
+                     accumulate)

@@ -1,8 +1,8 @@
 """One registry from an architecture's name to its model.
 
 A config.json names its architecture under ``architectures[0]`` (a class name such as
-``Qwen3ForCausalLM``), ``model_type`` (``qwen3``) or ``architecture`` (``Datasun``, ``Bepilorn``, ``Munerax``, ``Kikelorn``).  Any of them selects the entry; the lookup is
-exact and case-sensitive, and an unknown name is answered with the list of known ones, as in
+``Qwen3ForCausalLM``), ``model_type`` (``qwen3``) or ``architecture`` (``Datasun``, ``Bepilorn``, ``Munerax``, ``Kikelorn``,
+``Zirivik``).  Any of them selects the entry; the lookup is exact and case-sensitive, and an unknown name is answered with the list of known ones, as in
 the reference (crates/bfi-models/src/arch.rs:70-91).
 """
 from __future__ import annotations
@@ -82,6 +82,10 @@ def _register_builtin() -> None:
     from .config.kikelorn import KikelornConfig
     register_architecture(("Kikelorn", "kikelorn"),
                           Architecture(name="kikelorn", config_class=KikelornConfig, describe=kikelorn.describe))
+    from .architectures import zirivik
+    from .config.zirivik import ZirivikConfig
+    register_architecture(("Zirivik", "zirivik"),
+                          Architecture(name="zirivik", config_class=ZirivikConfig, describe=zirivik.describe))
 
 
 _register_builtin()
