@@ -9,6 +9,11 @@
 // They are merged in range order by a second kernel (which, launched as a programmatic dependent,
 // is already resident when the first one ends).
 //
+// Beside a window the first `keep_first` positions stay readable: the list of pages a sequence reads is
+// then the pages of those positions that lie before the window's first page, followed by the window's.
+// `split_p`: the weights enter the second product as two bfloat16 terms (the rounded weight and what the
+// rounding left over), float32 in effect.
+//
 // Scores, the running maximum and sum, and the output accumulator are float32; exp is
 // ex2.approx on scores pre-multiplied by log2(e).
 //
@@ -16,6 +21,20 @@
 // status word, the block gives its outstanding copies a bounded time to land and returns.
 #include "attention_tiles.cuh"
 #include "tcgen05.cuh"
+
+// The pages the token at `pos` reads, as a list: entry i is page i for i < n_keep, else page i + skip.
+struct DecodePages {
+    int lo, n_keep, skip, n_pages;
+};
+__device__ __forceinline__ DecodePages decode_pages(int pos, int window, int keep_first) {
+    DecodePages d;
+    d.lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int first = d.lo / AD_TILE;
+    d.n_keep = min((keep_first + AD_TILE - 1) / AD_TILE, first);
+    d.skip = first - d.n_keep;
+    d.n_pages = d.n_keep + pos / AD_TILE - first + 1;
+    return d;
+}
 
 // A sequence's pages are cut into at most `max_splits` ranges of equal size (in pages), so every
 // sequence, long or short, spreads over the same number of blocks.
@@ -44,12 +63,12 @@ struct DecodeSmem {
 
 // part_o  [seqs, n_q, max_splits, D]  float32 unnormalised outputs
 // part_ml [seqs, n_q, max_splits, 2]  float32 (running max in log2 units, running sum)
-template <int D>
+template <int D, bool SPLIT_P>
 __global__ void __launch_bounds__(AD_THREADS)
 attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out, long out_stride,
                         const int* __restrict__ block_table, int table_stride, const int* __restrict__ seq_slot,
-                        const int* __restrict__ seq_start, int n_q, int n_kv, int window, float scale_log2, float sink_log2,
+                        const int* __restrict__ seq_start, int n_q, int n_kv, int window, int keep_first, float scale_log2, float sink_log2,
                         int head_chunks, float* __restrict__ part_o, float* __restrict__ part_ml,
                         int* __restrict__ status, TcWaits waits) {
     pdl_trigger();
@@ -71,16 +90,16 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int g = lane >> 2, t = lane & 3;
 
-    const int pos = seq_start[seq];                       // the new token's position; keys lo..pos
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
-    const int first_page = lo / AD_TILE, last_page = pos / AD_TILE;
-    const int n_pages = last_page - first_page + 1;
+    const int pos = seq_start[seq];                       // the new token's position; keys lo..pos and the kept first ones
+    const DecodePages pages = decode_pages(pos, window, keep_first);
+    const int lo = pages.lo, n_pages = pages.n_pages;
     const int pages_per_split = decode_pages_per_split(n_pages, max_splits);
     const int n_splits = (n_pages + pages_per_split - 1) / pages_per_split;    // ranges this sequence has
     if (split >= n_splits) return;
-    const int p_beg = first_page + split * pages_per_split;
-    const int p_end = min(last_page + 1, p_beg + pages_per_split);
-    const int n_tiles = p_end - p_beg;
+    const int i_beg = split * pages_per_split;            // entries i_beg .. i_end-1 of the list are this block's
+    const int i_end = min(n_pages, i_beg + pages_per_split);
+    const int n_tiles = i_end - i_beg;
+    auto page_at = [&](int it) { return i_beg + it < pages.n_keep ? i_beg + it : i_beg + it + pages.skip; };
 
     const int* table = block_table + (size_t)slot * table_stride;
     if (threadIdx.x == 0) {
@@ -114,13 +133,13 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     int issued = 0;                                       // tiles on their way (thread 0 keeps count)
     const bool producer = threadIdx.x == 0 && !waits.hold_producer;
     if (producer)
-        while (issued < 2 && issued < n_tiles && p_beg + issued != last_page) {
-            issue(p_beg + issued, issued);
+        while (issued < 2 && issued < n_tiles && i_beg + issued != n_pages - 1) {
+            issue(page_at(issued), issued);
             ++issued;
         }
     pdl_wait();
     if (producer && issued == 0 && n_tiles > 0) {
-        issue(p_beg, 0);
+        issue(page_at(0), 0);
         issued = 1;
     }
 
@@ -151,11 +170,11 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 
     bool ok = true;
     for (int it = 0; it < n_tiles; ++it) {
-        const int p = p_beg + it;
+        const int p = page_at(it);
         const int stage = it & 1;
         // the other stage was read for the last time before the barrier that ended the iteration before
         if (producer && it + 1 < n_tiles && it + 1 >= issued) {
-            issue(p + 1, stage ^ 1);
+            issue(page_at(it + 1), stage ^ 1);
             ++issued;
         }
         ok = __syncthreads_and(mbar_wait(&full[stage], (uint32_t)((it >> 1) & 1), spin_limit));
@@ -215,7 +234,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 for (int c = 0; c < 2; ++c) {
                     const int key = key0 + j * 8 + 2 * t + c;
                     float v = s[j][r * 2 + c] * scale_log2;
-                    if (!have_page || key > pos || key < lo) v = -INFINITY;
+                    if (!have_page || key > pos || (key < lo && key >= keep_first)) v = -INFINITY;
                     s[j][r * 2 + c] = v;
                     mx = fmaxf(mx, v);
                 }
@@ -244,11 +263,17 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             }
         }
         // ---- P (16 heads x 16 keys) as the A operand, V rows of these 16 keys as B
-        uint32_t pa[4];
+        uint32_t pa[4], pl[4];
         pa[0] = pack_bf16(p_frag[0][0], p_frag[0][1]);
         pa[1] = pack_bf16(p_frag[0][2], p_frag[0][3]);
         pa[2] = pack_bf16(p_frag[1][0], p_frag[1][1]);
         pa[3] = pack_bf16(p_frag[1][2], p_frag[1][3]);
+        if (SPLIT_P) {
+            pl[0] = pack_bf16(p_frag[0][0] - bf16_lo(pa[0]), p_frag[0][1] - bf16_hi(pa[0]));
+            pl[1] = pack_bf16(p_frag[0][2] - bf16_lo(pa[1]), p_frag[0][3] - bf16_hi(pa[1]));
+            pl[2] = pack_bf16(p_frag[1][0] - bf16_lo(pa[2]), p_frag[1][1] - bf16_hi(pa[2]));
+            pl[3] = pack_bf16(p_frag[1][2] - bf16_lo(pa[3]), p_frag[1][3] - bf16_hi(pa[3]));
+        }
         if (have_page) {
 #pragma unroll
             for (int dd = 0; dd < D / 8; dd += 2) {
@@ -257,6 +282,10 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
                 ldmatrix_x4_trans(b, box_chunk<D>(vt, row, dd + (lane >> 4)));
                 mma16816(o[dd], pa, b[0], b[1]);
                 mma16816(o[dd + 1], pa, b[2], b[3]);
+                if (SPLIT_P) {
+                    mma16816(o[dd], pl, b[0], b[1]);
+                    mma16816(o[dd + 1], pl, b[2], b[3]);
+                }
             }
         }
         __syncthreads();      // the stage is free for the load issued in the next iteration
@@ -331,15 +360,14 @@ template <int D, int CAP>
 __global__ void attention_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                               const int* __restrict__ seq_slot, const int* __restrict__ seq_start,
                                               bf16* __restrict__ out, long out_stride, int n_q, int max_splits, int window,
-                                              float sink_log2) {
+                                              int keep_first, float sink_log2) {
     pdl_trigger();
     const int seq = blockIdx.y, head = blockIdx.x;
     const int slot = seq_slot[seq];
     const int pos = seq_start[seq];
     pdl_wait();
     if (slot < 0) return;
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
-    const int n_pages = pos / AD_TILE - lo / AD_TILE + 1;
+    const int n_pages = decode_pages(pos, window, keep_first).n_pages;
     const int pps = decode_pages_per_split(n_pages, max_splits);
     const int n_splits = (n_pages + pps - 1) / pps;
     if (n_splits == 1) return;                            // the first kernel wrote the output itself
@@ -370,8 +398,8 @@ __global__ void attention_decode_merge_kernel(const float* __restrict__ part_o, 
 template <int D>
 static int launch_decode(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                          const void* v_pages, long n_pages, const int* block_table, int table_stride,
-                         const int* seq_slot, const int* seq_start, int n_seqs, int n_q, int n_kv, int window, float scale,
-                         float sink, int max_splits, float* part_o, float* part_ml, int* status, cudaStream_t stream, TcWaits waits) {
+                         const int* seq_slot, const int* seq_start, int n_seqs, int n_q, int n_kv, int window, int keep_first,
+                         float scale, float sink, int split_p, int max_splits, float* part_o, float* part_ml, int* status, cudaStream_t stream, TcWaits waits) {
     CUtensorMap mk, mv;
     int rc = bfi_tensor_map_bf16(k_pages, n_pages * n_kv * AD_TILE, D, D, AD_TILE, &mk);
     if (rc) return rc;
@@ -380,7 +408,7 @@ static int launch_decode(const void* q, long q_stride, void* out, long out_strid
     const int group = n_q / n_kv;
     const int head_chunks = (group + 15) / 16;
     const size_t need = DecodeSmem<D>::BYTES;
-    auto kernel = attention_decode_kernel<D>;
+    auto kernel = split_p ? attention_decode_kernel<D, true> : attention_decode_kernel<D, false>;
     if (need > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)need);
         if (e != cudaSuccess) return bfi_fail("attention_decode: cannot reserve %zu bytes of shared memory: %s", need,
@@ -390,13 +418,13 @@ static int launch_decode(const void* q, long q_stride, void* out, long out_strid
     const float scale_log2 = scale * 1.4426950408889634f;
     const float sink_log2 = sink * 1.4426950408889634f;       // -inf: no sink
     bfi_launch(kernel, grid, dim3(AD_THREADS), need, stream, mk, mv, (const bf16*)q, q_stride, (bf16*)out, out_stride,
-               block_table, table_stride, seq_slot, seq_start, n_q, n_kv, window, scale_log2, sink_log2, head_chunks, part_o, part_ml,
+               block_table, table_stride, seq_slot, seq_start, n_q, n_kv, window, keep_first, scale_log2, sink_log2, head_chunks, part_o, part_ml,
                status, waits);
     rc = bfi_check_launch("attention_decode");
     if (rc || max_splits == 1) return rc;
 #define BFI_MERGE(CAP)                                                                                                   \
     bfi_launch(attention_decode_merge_kernel<D, CAP>, dim3(n_q, n_seqs), dim3(D), 0, stream, (const float*)part_o,        \
-               (const float*)part_ml, seq_slot, seq_start, (bf16*)out, out_stride, n_q, max_splits, window, sink_log2)
+               (const float*)part_ml, seq_slot, seq_start, (bf16*)out, out_stride, n_q, max_splits, window, keep_first, sink_log2)
     if (max_splits <= 8) BFI_MERGE(8);
     else if (max_splits <= 16) BFI_MERGE(16);
     else BFI_MERGE(32);
@@ -413,10 +441,11 @@ static int launch_decode(const void* q, long q_stride, void* out, long out_strid
 static int attention_decode_launch(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                                    const void* v_pages, long n_pages, const int* block_table, int table_stride,
                                    const int* seq_slot, const int* seq_start, int n_seqs, int n_q, int n_kv, int d,
-                                   int window, float scale, float sink, int max_splits, float* part_o, float* part_ml,
-                                   int* status, cudaStream_t stream, TcWaits waits) {
+                                   int window, int keep_first, float scale, float sink, int split_p, int max_splits, float* part_o,
+                                   float* part_ml, int* status, cudaStream_t stream, TcWaits waits) {
     BFI_REQUIRE(n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_decode: %d query heads do not divide into %d kv heads",
                 n_q, n_kv);
+    BFI_REQUIRE(keep_first == 0 || (keep_first > 0 && window > 0), "attention_decode: first positions are kept beside a window");
     BFI_REQUIRE(window >= 0 && max_splits >= 1 && max_splits <= 32, "attention_decode: bad window or split count (1..32)");
     BFI_REQUIRE(status != nullptr && n_pages > 0, "attention_decode: no status word or no pages");
     if (n_seqs <= 0) return 0;
@@ -426,21 +455,21 @@ static int attention_decode_launch(const void* q, long q_stride, void* out, long
     if (max_splits > 1) BFI_REQUIRE(part_o && part_ml, "attention_decode: split runs need the scratch buffers");
     if (d == 64)
         return launch_decode<64>(q, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
-                                 seq_slot, seq_start, n_seqs, n_q, n_kv, window, scale, sink, max_splits, part_o, part_ml, status,
-                                 stream, waits);
+                                 seq_slot, seq_start, n_seqs, n_q, n_kv, window, keep_first, scale, sink, split_p, max_splits, part_o, part_ml,
+                                 status, stream, waits);
     return launch_decode<128>(q, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride, seq_slot,
-                              seq_start, n_seqs, n_q, n_kv, window, scale, sink, max_splits, part_o, part_ml, status, stream,
-                              waits);
+                              seq_start, n_seqs, n_q, n_kv, window, keep_first, scale, sink, split_p, max_splits, part_o, part_ml, status,
+                              stream, waits);
 }
 
 extern "C" int bfi_attention_decode_bf16(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                                          const void* v_pages, long n_pages, const int* block_table, int table_stride,
                                          const int* seq_slot, const int* seq_start, int n_seqs, int n_q, int n_kv,
-                                         int d, int window, float scale, float sink, int max_splits, float* part_o,
-                                         float* part_ml, int* status, cudaStream_t stream) {
+                                         int d, int window, int keep_first, float scale, float sink, int split_p,
+                                         int max_splits, float* part_o, float* part_ml, int* status, cudaStream_t stream) {
     return attention_decode_launch(q, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
-                                   seq_slot, seq_start, n_seqs, n_q, n_kv, d, window, scale, sink, max_splits, part_o, part_ml,
-                                   status, stream, tc_waits_default());
+                                   seq_slot, seq_start, n_seqs, n_q, n_kv, d, window, keep_first, scale, sink, split_p, max_splits, part_o,
+                                   part_ml, status, stream, tc_waits_default());
 }
 
 // The same launch with its bounded waits cut to `spin_limit` polls and, with hold_producer, a thread
@@ -456,7 +485,7 @@ extern "C" int bfi_attention_decode_bf16_wait_probe(const void* q, long q_stride
                                                     cudaStream_t stream) {
     BFI_REQUIRE(spin_limit > 0 && spin_limit <= TC_SPIN_LIMIT, "attention_decode probe: spin limit out of range");
     return attention_decode_launch(q, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
-                                   seq_slot, seq_start, n_seqs, n_q, n_kv, d, window, scale, -INFINITY, max_splits, part_o, part_ml,
+                                   seq_slot, seq_start, n_seqs, n_q, n_kv, d, window, 0, scale, -INFINITY, 0, max_splits, part_o, part_ml,
                                    status, stream, TcWaits{spin_limit, hold_producer ? 1 : 0});
 }
 

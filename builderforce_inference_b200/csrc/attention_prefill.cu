@@ -1,6 +1,7 @@
 // Prompt attention for bfloat16 on the tensor cores: every new token of a step attends causally
 // over the cached keys and values of its sequence (the step's own tokens are already in the cache),
-// whole prompts and continuations of a cached prefix alike, with an optional window
+// whole prompts and continuations of a cached prefix alike, with an optional window (beside which the
+// sequence's first `keep_first` positions may stay readable: their pages come first, then the window's)
 // (crates/bfi-core/src/cpu.rs:328-392).
 //
 // One block per (sequence, query head, 64 consecutive tokens); each of its four warps owns 16
@@ -19,7 +20,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __rest
                          const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                          const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_seqlens,
                          const int* __restrict__ seq_slot, const int* __restrict__ seq_start, int n_q, int n_kv,
-                         int window, int chunk, float scale_log2, float sink_log2, const float* __restrict__ sinks,
+                         int window, int keep_first, int chunk, float scale_log2, float sink_log2, const float* __restrict__ sinks,
                          int split_p) {
     pdl_trigger();
     pdl_wait();
@@ -46,6 +47,9 @@ attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __rest
     int lo_block = window > 0 ? max(0, start + tok0 - window + 1) : 0;
     if (chunk > 0) lo_block = max(lo_block, (start + tok0) / chunk * chunk);     // a token reads its own chunk of positions only
     const int p_beg = lo_block / AD_TILE, p_end = hi_block / AD_TILE;    // inclusive
+    const int n_keep = min((keep_first + AD_TILE - 1) / AD_TILE, p_beg); // pages of kept positions before them
+    const int n_list = n_keep + p_end - p_beg + 1;
+    auto page_at = [&](int i) { return i < n_keep ? i : p_beg + i - n_keep; };
 
     // ---- Q tile -> shared memory (rows past the sequence are zero)
     {
@@ -70,7 +74,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __rest
         }
         cp_async_commit();
     };
-    issue(p_beg, 0);                     // the Q copies ride in this first group
+    issue(page_at(0), 0);                // the Q copies ride in this first group
 
     // rows of this warp: tokens tok0 + 16*warp + g and + 8
     int pos_r[2], lo_r[2];
@@ -96,16 +100,17 @@ attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __rest
 #pragma unroll
         for (int j = 0; j < 4; ++j) o[i][j] = 0.0f;
 
-    for (int p = p_beg; p <= p_end; ++p) {
-        const int stage = (p - p_beg) & 1;
-        if (p + 1 <= p_end) {
-            issue(p + 1, stage ^ 1);
+    for (int i_page = 0; i_page < n_list; ++i_page) {
+        const int p = page_at(i_page);
+        const int stage = i_page & 1;
+        if (i_page + 1 < n_list) {
+            issue(page_at(i_page + 1), stage ^ 1);
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
         }
         __syncthreads();
-        if (p == p_beg) {
+        if (i_page == 0) {
             // query fragments: 16 rows of this warp, all of D
 #pragma unroll
             for (int kk = 0; kk < D / 16; ++kk) {
@@ -128,7 +133,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __rest
             __syncthreads();
         }
         const int key_lo = p * AD_TILE, key_hi = key_lo + AD_TILE - 1;
-        if (have_page && key_lo <= warp_pos_max && key_hi >= warp_lo_min) {
+        if (have_page && key_lo <= warp_pos_max && (key_hi >= warp_lo_min || key_lo < keep_first)) {
             // ---- scores: 16 tokens x 64 keys
             float s[8][4];
 #pragma unroll
@@ -157,7 +162,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __rest
                         float v = s[j][r * 2 + c] * scale_log2;
                         if (need_mask) {
                             const int key = key_lo + j * 8 + 2 * t + c;
-                            if (key > pos_r[r] || key < lo_r[r]) v = -INFINITY;
+                            if (key > pos_r[r] || (key < lo_r[r] && key >= keep_first)) v = -INFINITY;
                         }
                         s[j][r * 2 + c] = v;
                         mx = fmaxf(mx, v);
@@ -241,7 +246,7 @@ template <int D>
 static int launch_prefill(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                           const void* v_pages, const int* block_table, int table_stride, const int* cu_seqlens,
                           const int* seq_slot, const int* seq_start, int n_seqs, int max_tokens, int n_q, int n_kv,
-                          int window, int chunk, float scale, float sink, const float* sinks, int split_p,
+                          int window, int keep_first, int chunk, float scale, float sink, const float* sinks, int split_p,
                           cudaStream_t stream) {
     const size_t smem = (size_t)(AP_QROWS * D + 4 * AD_TILE * D) * sizeof(bf16);
     auto kernel = attention_prefill_kernel<D>;
@@ -253,7 +258,7 @@ static int launch_prefill(const void* q, long q_stride, void* out, long out_stri
     dim3 grid((max_tokens + AP_QROWS - 1) / AP_QROWS, n_q, n_seqs);
     bfi_launch(kernel, grid, dim3(AD_THREADS), smem, stream, (const bf16*)q, q_stride, (bf16*)out, out_stride,
                (const bf16*)k_pages, (const bf16*)v_pages, block_table, table_stride, cu_seqlens, seq_slot, seq_start, n_q,
-               n_kv, window, chunk, scale * 1.4426950408889634f, sink * 1.4426950408889634f, sinks, split_p);
+               n_kv, window, keep_first, chunk, scale * 1.4426950408889634f, sink * 1.4426950408889634f, sinks, split_p);
     return bfi_check_launch("attention_prefill");
 }
 
@@ -266,11 +271,12 @@ static int launch_prefill(const void* q, long q_stride, void* out, long out_stri
 extern "C" int bfi_attention_prefill_bf16(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                                           const void* v_pages, const int* block_table, int table_stride,
                                           const int* cu_seqlens, const int* seq_slot, const int* seq_start, int n_seqs,
-                                          int max_tokens, int n_q, int n_kv, int d, int window, int chunk, float scale,
+                                          int max_tokens, int n_q, int n_kv, int d, int window, int keep_first, int chunk, float scale,
                                           float sink, const float* sinks, int split_p, cudaStream_t stream) {
     BFI_REQUIRE(n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_prefill: %d query heads do not divide into %d kv heads",
                 n_q, n_kv);
     BFI_REQUIRE(window >= 0 && chunk >= 0, "attention_prefill: negative window or chunk");
+    BFI_REQUIRE(keep_first == 0 || (keep_first > 0 && window > 0 && chunk == 0), "attention_prefill: first positions are kept beside a window");
     if (n_seqs <= 0 || max_tokens <= 0) return 0;
     if (d != 64 && d != 128) return 2;
     if (q_stride % 8 != 0 || out_stride % 2 != 0 || ((uintptr_t)q & 15) || ((uintptr_t)out & 3) || n_seqs > 65535 ||
@@ -278,9 +284,9 @@ extern "C" int bfi_attention_prefill_bf16(const void* q, long q_stride, void* ou
         return 2;
     if (d == 64)
         return launch_prefill<64>(q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride, cu_seqlens,
-                                  seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, window, chunk, scale, sink, sinks, split_p,
+                                  seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, window, keep_first, chunk, scale, sink, sinks, split_p,
                                   stream);
     return launch_prefill<128>(q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride, cu_seqlens,
-                               seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, window, chunk, scale, sink, sinks, split_p,
+                               seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, window, keep_first, chunk, scale, sink, sinks, split_p,
                                stream);
 }

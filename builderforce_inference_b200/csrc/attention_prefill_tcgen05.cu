@@ -1,6 +1,8 @@
 // Prompt attention for bfloat16 on the fifth-generation tensor cores: every new token of a step
 // attends causally over the cached keys and values of its sequence (the step's own tokens are
-// already in the cache), with an optional window (crates/bfi-core/src/cpu.rs:328-392).
+// already in the cache), with an optional window (crates/bfi-core/src/cpu.rs:328-392), beside which the
+// sequence's first `keep_first` positions may stay readable: an item's tiles are then the tiles of those
+// positions that lie before its window, followed by the window's.
 //
 // A work item is (sequence, query head, 128 consecutive tokens).  One block per SM draws items
 // from a shared ticket counter until none is left: the token tiles from the last one down (the
@@ -14,6 +16,9 @@
 //                (one lane per token, one column per key), double-buffered
 //   O += P V     P (bfloat16) read from tensor memory, where the softmax wrote it over S;
 //                V [128 keys x D] from shared memory as the MN-major operand
+//
+// SPLIT_P: the weights are float32 in effect.  What the rounding of P to bfloat16 left over is a second
+// bfloat16 operand in the other half of the S buffer's columns, with a product of its own.
 //
 //   warps 0-3  softmax: thread r owns token r.  It reads its row of S (tcgen05.ld), masks it on
 //              tiles that touch the diagonal, the window's edge or the sequence's end, and writes
@@ -166,16 +171,16 @@ struct FtItem {
     int row0;         // row of the item's first token in q and out
     int rows;         // tokens of the item that exist (at most FT_ROWS)
     int head;
-    int pad;
+    int n_keep;       // tiles of kept first positions at the head of the list: tile i is i for i < n_keep, else j_beg + i - n_keep
 };
 
-template <int D>
+template <int D, bool SPLIT_P>
 __global__ void __launch_bounds__(FT_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, long out_stride,
                             const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_seqlens,
                             const int* __restrict__ seq_slot, const int* __restrict__ seq_start, int n_seqs, int max_tiles,
-                            int n_q, int n_kv, int window, float scale_log2, float sink_log2, uint32_t v_lbo, uint32_t v_sbo,
+                            int n_q, int n_kv, int window, int keep_first, float scale_log2, float sink_log2, uint32_t v_lbo, uint32_t v_sbo,
                             int* __restrict__ status, int* __restrict__ counters, TcWaits waits) {
     const uint32_t spin_limit = waits.spin_limit;
     constexpr int BOXES = D / 64;
@@ -265,7 +270,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         // share; an item is prepared (its sequence's numbers, the page ids of its first key tile)
         // while the last tiles of the item before it are loaded.
         struct Prep {
-            int have, head, kvh, tok0, slot, t0, nt, start, j_beg, n_tiles, pg0, pg1;
+            int have, head, kvh, tok0, slot, t0, nt, start, j_beg, n_keep, n_tiles, pg0, pg1;
         };
         int drawn = 0;                                     // lane 0: the ticket drawn last
         auto draw = [&]() {
@@ -292,9 +297,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 const int hi_block = p.start + min(p.tok0 + FT_ROWS - 1, p.nt - 1);
                 const int lo_block = window > 0 ? max(0, p0 - window + 1) : 0;
                 p.j_beg = lo_block / FT_KEYS;
-                p.n_tiles = hi_block / FT_KEYS - p.j_beg + 1;                          // key tiles
-                p.pg0 = page_of(p.slot, 2 * p.j_beg);
-                p.pg1 = page_of(p.slot, 2 * p.j_beg + 1);
+                p.n_keep = min((keep_first + FT_KEYS - 1) / FT_KEYS, p.j_beg);
+                p.n_tiles = p.n_keep + hi_block / FT_KEYS - p.j_beg + 1;               // key tiles
+                const int j0 = p.n_keep > 0 ? 0 : p.j_beg;
+                p.pg0 = page_of(p.slot, 2 * j0);
+                p.pg1 = page_of(p.slot, 2 * j0 + 1);
                 return p;
             }
         };
@@ -316,6 +323,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     items[qi].row0 = p.t0 + p.tok0;
                     items[qi].rows = p.nt - p.tok0;
                     items[qi].head = p.head;
+                    items[qi].n_keep = p.n_keep;
                     mbar_expect_tx(&q_full[qi], TILE_BYTES);
                     for (int c = 0; c < BOXES; ++c)
                         tma_load_2d(q_smem + (size_t)qi * TILE_BYTES + c * FT_BOX_BYTES, &map_q, p.head * D + c * 64,
@@ -330,16 +338,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         bool failed = !announce(0, cur);
         for (int it = 0; !failed && cur.have; ++it, cur = nxt) {
             int ok = 1;
-            const int kvh = cur.kvh, slot = cur.slot, j_beg = cur.j_beg, n_tiles = cur.n_tiles;
+            const int kvh = cur.kvh, slot = cur.slot, j_beg = cur.j_beg, n_keep = cur.n_keep, n_tiles = cur.n_tiles;
             const int seq_hi = cur.start + cur.nt - 1;                          // last position the cache holds
             int pg_next[2] = {cur.pg0, cur.pg1};
             for (int i = 0; i < n_tiles; ++i, ++g) {
-                const int j = j_beg + i, st = g & 1;
+                const int j = i < n_keep ? i : j_beg + i - n_keep, st = g & 1;
                 const uint32_t ph = (g >> 1) & 1;
                 const int pg[2] = {pg_next[0], pg_next[1]};
                 if (i + 1 < n_tiles) {                     // the next tile's page ids travel while this tile is handled
-                    pg_next[0] = page_of(slot, 2 * j + 2);
-                    pg_next[1] = page_of(slot, 2 * j + 3);
+                    const int jn = i + 1 < n_keep ? i + 1 : j_beg + i + 1 - n_keep;
+                    pg_next[0] = page_of(slot, 2 * jn);
+                    pg_next[1] = page_of(slot, 2 * jn + 1);
                 }
                 const int n_have = (pg[0] >= 0) + (pg[1] >= 0);
                 unsigned char* kt = k_smem + (size_t)st * TILE_BYTES;
@@ -472,6 +481,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                     for (int kk = 0; kk < FT_KEYS / 16; ++kk)       // 16 keys per step: 8 columns of packed P, 2048 bytes of V
                         umma_bf16_a_tmem(o_addr, p_addr + kk * 8, vd + (uint64_t)(kk * 2048 >> 4), idesc_o, (i > 0 || kk > 0));
+                    if (SPLIT_P) {
+#pragma unroll
+                        for (int kk = 0; kk < FT_KEYS / 16; ++kk)
+                            umma_bf16_a_tmem(o_addr, p_addr + FT_KEYS / 2 + kk * 8, vd + (uint64_t)(kk * 2048 >> 4), idesc_o, 1u);
+                    }
                     umma_commit(&v_empty[b]);
                     umma_commit(o_tile);
                     if (i + 1 == n_cur) umma_commit(&o_done[qi]);
@@ -506,7 +520,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             const int qi = it & 1;
             if (!__all_sync(FULL, MBAR_WAIT(&q_full[qi], (uint32_t)(it >> 1) & 1))) { ok = false; timed_out = true; break; }
             const int n_tiles = items[qi].n_tiles, j_beg = items[qi].j_beg, p0 = items[qi].p0, seq_hi = items[qi].seq_hi;
-            const int row0 = items[qi].row0, rows = items[qi].rows, head = items[qi].head;
+            const int row0 = items[qi].row0, rows = items[qi].rows, head = items[qi].head, n_keep = items[qi].n_keep;
             __syncwarp();
             if (lane == 0) mbar_arrive(&q_empty[qi]);
             if (n_tiles == 0) break;
@@ -516,7 +530,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             float m_used = -INFINITY, l_run = 0.0f;
             for (int i = 0; i < n_tiles; ++i, ++g) {
                 if (__any_sync(FULL, *s_flag != 0)) { ok = false; break; }
-                const int j = j_beg + i;
+                const int j = i < n_keep ? i : j_beg + i - n_keep;
                 const uint32_t b = g & 1, ph = (g >> 1) & 1;
                 if (!__all_sync(FULL, MBAR_WAIT(&s_full[b], ph))) { ok = false; timed_out = true; break; }
                 tc_fence_after();
@@ -531,12 +545,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 if (masked) {
                     // keep lo <= index <= hi; by groups of 32 keys, so that a warp passes over the
                     // groups that all its rows keep whole (on the diagonal: those left of its rows)
-                    const int hi = pos_r - key0, lo = lo_r - key0;
+                    const int hi = pos_r - key0, lo = lo_r - key0, keep = keep_first - key0;     // ... or index < keep
 #pragma unroll
                     for (int c = 0; c < FT_KEYS / 32; ++c) {
-                        if (__all_sync(FULL, c * 32 + 31 <= hi && c * 32 >= lo)) continue;
+                        if (__all_sync(FULL, c * 32 + 31 <= hi && (c * 32 >= lo || c * 32 + 31 < keep))) continue;
 #pragma unroll
-                        for (int e = c * 32; e < c * 32 + 32; ++e) s[e] = (e > hi || e < lo) ? -INFINITY : s[e];
+                        for (int e = c * 32; e < c * 32 + 32; ++e) s[e] = (e > hi || (e < lo && e >= keep)) ? -INFINITY : s[e];
                     }
                 }
                 float mx = s[0];
@@ -570,17 +584,36 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 }
                 const float mc = m_used == -INFINITY ? 0.0f : m_used * scale_log2;
                 float sum = 0.0f;
-                uint32_t pk[FT_KEYS / 2];
+                if (SPLIT_P) {
+                    // 64 keys at a time, so that the two terms fit beside the scores still to come
 #pragma unroll
-                for (int e = 0; e < FT_KEYS; e += 2) {
-                    const float a = ft_exp2(fmaf(s[e], scale_log2, -mc));
-                    const float c2 = ft_exp2(fmaf(s[e + 1], scale_log2, -mc));
-                    sum += a + c2;
-                    pk[e >> 1] = ft_pack(a, c2);
+                    for (int c = 0; c < FT_KEYS / 64; ++c) {
+                        uint32_t pk[32], pl[32];
+#pragma unroll
+                        for (int e = 0; e < 64; e += 2) {
+                            const float a = ft_exp2(fmaf(s[c * 64 + e], scale_log2, -mc));
+                            const float c2 = ft_exp2(fmaf(s[c * 64 + e + 1], scale_log2, -mc));
+                            sum += a + c2;
+                            const uint32_t p2 = ft_pack(a, c2);
+                            pk[e >> 1] = p2;
+                            pl[e >> 1] = ft_pack(a - __uint_as_float(p2 << 16), c2 - __uint_as_float(p2 & 0xffff0000u));
+                        }
+                        tmem_st32(s_addr + c * 32, pk);
+                        tmem_st32(s_addr + FT_KEYS / 2 + c * 32, pl);
+                    }
+                } else {
+                    uint32_t pk[FT_KEYS / 2];
+#pragma unroll
+                    for (int e = 0; e < FT_KEYS; e += 2) {
+                        const float a = ft_exp2(fmaf(s[e], scale_log2, -mc));
+                        const float c2 = ft_exp2(fmaf(s[e + 1], scale_log2, -mc));
+                        sum += a + c2;
+                        pk[e >> 1] = ft_pack(a, c2);
+                    }
+#pragma unroll
+                    for (int c = 0; c < FT_KEYS / 64; ++c) tmem_st32(s_addr + c * 32, pk + c * 32);
                 }
                 l_run += sum;
-#pragma unroll
-                for (int c = 0; c < FT_KEYS / 64; ++c) tmem_st32(s_addr + c * 32, pk + c * 32);
                 tmem_wait_st();
                 tc_fence_before();
                 mbar_arrive(&p_full[b]);
@@ -630,11 +663,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     BFI_TRACE_END();
 }
 
-template <int D>
+template <int D, bool SPLIT_P>
 static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out_stride, const void* k_pages,
                              const void* v_pages, long n_pages, const int* block_table, int table_stride,
                              const int* cu_seqlens, const int* seq_slot, const int* seq_start, int n_seqs, long n_tokens,
-                             int max_seq_tokens, int n_q, int n_kv, int window, float scale, float sink, int* status,
+                             int max_seq_tokens, int n_q, int n_kv, int window, int keep_first, float scale, float sink, int* status,
                              cudaStream_t stream, TcWaits waits) {
     CUtensorMap mq, mk, mv;
     int rc = bfi_tensor_map_bf16(qkv, n_tokens, (long)n_q * D, q_stride, FT_ROWS, &mq);
@@ -647,7 +680,7 @@ static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out
     // at least half an SM's shared memory, so that two blocks never share one SM's tensor memory
     const size_t tiles = (size_t)6 * TILE_BYTES + 1024 + 512 + FT_META_SEQS * sizeof(int4) + 4 * 4096;
     const size_t smem = tiles > 120 * 1024 ? tiles : 120 * 1024;
-    auto kernel = attention_prefill_tc_kernel<D>;
+    auto kernel = attention_prefill_tc_kernel<D, SPLIT_P>;
     static bool configured = false;
     const int n_sm = bfi_sm_count();
     if (!configured) {
@@ -662,7 +695,7 @@ static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out
     const long items = (long)max_tiles * n_seqs * n_q;
     dim3 grid((unsigned)(items < n_sm ? items : n_sm));      // one block per SM, each drawing items until none is left
     bfi_launch(kernel, grid, dim3(FT_THREADS), smem, stream, mq, mk, mv, (bf16*)out, out_stride, block_table, table_stride,
-               cu_seqlens, seq_slot, seq_start, n_seqs, max_tiles, n_q, n_kv, window, scale * 1.4426950408889634f,
+               cu_seqlens, seq_slot, seq_start, n_seqs, max_tiles, n_q, n_kv, window, keep_first, scale * 1.4426950408889634f,
                sink * 1.4426950408889634f, (uint32_t)lbo, (uint32_t)sbo, status, status + 1, waits);
     return bfi_check_launch("attention_prefill_tcgen05");
 }
@@ -678,35 +711,38 @@ static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out
 static int attention_prefill_tc_launch(const void* qkv, long q_stride, void* out, long out_stride, const void* k_pages,
                                        const void* v_pages, long n_pages, const int* block_table, int table_stride,
                                        const int* cu_seqlens, const int* seq_slot, const int* seq_start, int n_seqs,
-                                       long n_tokens, int max_seq_tokens, int n_q, int n_kv, int d, int window, float scale,
-                                       float sink, int* status, cudaStream_t stream, TcWaits waits) {
+                                       long n_tokens, int max_seq_tokens, int n_q, int n_kv, int d, int window, int keep_first,
+                                       float scale, float sink, int split_p, int* status, cudaStream_t stream, TcWaits waits) {
     BFI_REQUIRE(n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_prefill_tcgen05: %d query heads do not divide into %d kv heads",
                 n_q, n_kv);
     BFI_REQUIRE(window >= 0 && status != nullptr, "attention_prefill_tcgen05: bad window or no status word");
+    BFI_REQUIRE(keep_first == 0 || (keep_first > 0 && window > 0), "attention_prefill_tcgen05: first positions are kept beside a window");
     if (n_seqs <= 0 || max_seq_tokens <= 0) return 0;
     if (d != 64 && d != 128) return 2;
     if (q_stride % 8 != 0 || out_stride % 8 != 0 || ((uintptr_t)qkv & 15) || ((uintptr_t)out & 15) ||
         ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15) || (long)((max_seq_tokens + FT_ROWS - 1) / FT_ROWS) * n_seqs * n_q > 0x3fffffffL)
         return 2;
     if (n_pages * n_kv * FT_PAGE > 0x7fffffffL) return 2;       // TMA coordinates are 32-bit
-    if (d == 64)
-        return launch_prefill_tc<64>(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
-                                     cu_seqlens, seq_slot, seq_start, n_seqs, n_tokens, max_seq_tokens, n_q, n_kv, window,
-                                     scale, sink, status, stream, waits);
-    return launch_prefill_tc<128>(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
-                                  cu_seqlens, seq_slot, seq_start, n_seqs, n_tokens, max_seq_tokens, n_q, n_kv, window, scale,
-                                  sink, status, stream, waits);
+#define BFI_PREFILL_TC(DD, SP)                                                                                              \
+    return launch_prefill_tc<DD, SP>(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,   \
+                                     cu_seqlens, seq_slot, seq_start, n_seqs, n_tokens, max_seq_tokens, n_q, n_kv, window,   \
+                                     keep_first, scale, sink, status, stream, waits)
+    if (d == 64 && split_p) BFI_PREFILL_TC(64, true);
+    if (d == 64) BFI_PREFILL_TC(64, false);
+    if (split_p) BFI_PREFILL_TC(128, true);
+    BFI_PREFILL_TC(128, false);
+#undef BFI_PREFILL_TC
 }
 
 extern "C" int bfi_attention_prefill_tcgen05_bf16(const void* qkv, long q_stride, void* out, long out_stride,
                                                   const void* k_pages, const void* v_pages, long n_pages,
                                                   const int* block_table, int table_stride, const int* cu_seqlens,
                                                   const int* seq_slot, const int* seq_start, int n_seqs, long n_tokens,
-                                                  int max_seq_tokens, int n_q, int n_kv, int d, int window, float scale,
-                                                  float sink, int* status, cudaStream_t stream) {
+                                                  int max_seq_tokens, int n_q, int n_kv, int d, int window, int keep_first,
+                                                  float scale, float sink, int split_p, int* status, cudaStream_t stream) {
     return attention_prefill_tc_launch(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
                                        cu_seqlens, seq_slot, seq_start, n_seqs, n_tokens, max_seq_tokens, n_q, n_kv, d, window,
-                                       scale, sink, status, stream, tc_waits_default());
+                                       keep_first, scale, sink, split_p, status, stream, tc_waits_default());
 }
 
 // For the tests of the time-out path: the same launch, but every bounded wait gives up after
@@ -726,7 +762,7 @@ extern "C" int bfi_attention_prefill_tcgen05_bf16_wait_probe(const void* qkv, lo
                 spin_limit);
     return attention_prefill_tc_launch(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
                                        cu_seqlens, seq_slot, seq_start, n_seqs, n_tokens, max_seq_tokens, n_q, n_kv, d, window,
-                                       scale, -INFINITY, status, stream, TcWaits{spin_limit, hold_producer ? 1 : 0});
+                                       0, scale, -INFINITY, 0, status, stream, TcWaits{spin_limit, hold_producer ? 1 : 0});
 }
 
 BFI_TRACE_EXPORT(attention_prefill_tcgen05)

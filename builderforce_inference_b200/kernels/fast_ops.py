@@ -188,9 +188,9 @@ def _sink(sink) -> c_float:
 
 
 def attention_decode_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads: int, scale: float,
-                          probe=None, sink=None) -> bool:
+                          probe=None, sink=None, exact_weights: bool = False) -> bool:
     """One new token per sequence over its cached pages, which arrive by TMA: the cache must be
-    contiguous.  A wait for a page that ran out shows in ``tc_status``.  ``probe``: (polls, hold
+    contiguous.  ``exact_weights``: as ``attention_prefill_bf16``.  A wait for a page that ran out shows in ``tc_status``.  ``probe``: (polls, hold
     the producer), for ``attention_decode_wait_probe``."""
     d = kv.head_dim
     if d not in (64, 128) or qkv.dtype != torch.bfloat16 or kv.k.dtype != torch.bfloat16:
@@ -202,7 +202,7 @@ def attention_decode_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads
     if bucket:
         max_pages = min(max_pages, bucket)           # what the step's sequences hold now, rounded up
     if kv.window:
-        max_pages = min(max_pages, (kv.window + 62) // 64 + 1)
+        max_pages = min(max_pages, (kv.window + 62) // 64 + 1 + (kv.keep_first + 63) // 64)
     group = n_heads // kv.n_kv_heads
     max_splits = decode_splits(ctx.n_seqs, kv.n_kv_heads, group, max_pages, sm_count(qkv.device))
     part_o = part_ml = None
@@ -211,12 +211,12 @@ def attention_decode_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads
         part_ml = ctx.workspace.vector("attn.part_ml", ctx.n_seqs * n_heads * max_splits * 2, torch.float32)
     args = [_ptr(qkv), c_long(qkv.stride(0)), _ptr(out), c_long(out.stride(0)), _ptr(kv.k), _ptr(kv.v),
             c_long(kv.k.shape[0]), _ptr(kv.block_table), c_int(kv.block_table.stride(0)), _ptr(ctx.seq_slot),
-            _ptr(ctx.seq_start), c_int(ctx.n_seqs), c_int(n_heads), c_int(kv.n_kv_heads), c_int(d), c_int(kv.window or 0),
-            c_float(scale)]
+            _ptr(ctx.seq_start), c_int(ctx.n_seqs), c_int(n_heads), c_int(kv.n_kv_heads), c_int(d), c_int(kv.window or 0)]
     tail = [c_int(max_splits), _ptr(part_o), _ptr(part_ml), _ptr(tc_status(qkv.device))]
     if probe is None:
-        return library("fast").call_optional("bfi_attention_decode_bf16", *args, _sink(sink), *tail, _stream())
-    args += tail
+        return library("fast").call_optional("bfi_attention_decode_bf16", *args, c_int(kv.keep_first), c_float(scale),
+                                             _sink(sink), c_int(1 if exact_weights else 0), *tail, _stream())
+    args += [c_float(scale)] + tail
     return library("fast").call_optional("bfi_attention_decode_bf16_wait_probe", *args, c_int(int(probe[0])),
                                          c_int(1 if probe[1] else 0), _stream())
 
@@ -240,7 +240,7 @@ def attention_prefill_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_head
         "bfi_attention_prefill_bf16", _ptr(qkv), c_long(qkv.stride(0)), _ptr(out), c_long(out.stride(0)), _ptr(kv.k),
         _ptr(kv.v), _ptr(kv.block_table), c_int(kv.block_table.stride(0)), _ptr(ctx.cu_seqlens), _ptr(ctx.seq_slot),
         _ptr(ctx.seq_start), c_int(ctx.n_seqs), c_int(ctx.max_seq_tokens), c_int(n_heads), c_int(kv.n_kv_heads),
-        c_int(d), c_int(kv.window or 0), c_int(kv.chunk or 0), c_float(scale), _sink(None if sinks is not None else sink),
+        c_int(d), c_int(kv.window or 0), c_int(kv.keep_first), c_int(kv.chunk or 0), c_float(scale), _sink(None if sinks is not None else sink),
         _ptr(sinks), c_int(1 if exact_weights else 0), _stream())
 
 
@@ -303,9 +303,10 @@ TCGEN05_ATTENTION_MIN_TOKENS = 128     # shorter steps: the mma.sync kernel with
 
 
 def attention_prefill_tcgen05_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads: int, scale: float,
-                                   sink=None) -> bool:
+                                   sink=None, exact_weights: bool = False) -> bool:
     """tcgen05 / TMA attention for steps with long runs of new tokens: one block per SM draws
-    items of 128 tokens of one head, scores and output in tensor memory.  A wait that ran out
+    items of 128 tokens of one head, scores and output in tensor memory.  ``exact_weights``: as
+    ``attention_prefill_bf16``.  A wait that ran out
     shows in ``tc_status``."""
     d = kv.head_dim
     if d not in (64, 128) or qkv.dtype != torch.bfloat16 or kv.k.dtype != torch.bfloat16:
@@ -316,8 +317,8 @@ def attention_prefill_tcgen05_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv
         "bfi_attention_prefill_tcgen05_bf16", _ptr(qkv), c_long(qkv.stride(0)), _ptr(out), c_long(out.stride(0)),
         _ptr(kv.k), _ptr(kv.v), c_long(kv.k.shape[0]), _ptr(kv.block_table), c_int(kv.block_table.stride(0)),
         _ptr(ctx.cu_seqlens), _ptr(ctx.seq_slot), _ptr(ctx.seq_start), c_int(ctx.n_seqs), c_long(qkv.shape[0]),
-        c_int(ctx.max_seq_tokens), c_int(n_heads), c_int(kv.n_kv_heads), c_int(d), c_int(kv.window or 0), c_float(scale),
-        _sink(sink), _ptr(tc_status(qkv.device)), _stream())
+        c_int(ctx.max_seq_tokens), c_int(n_heads), c_int(kv.n_kv_heads), c_int(d), c_int(kv.window or 0),
+        c_int(kv.keep_first), c_float(scale), _sink(sink), c_int(1 if exact_weights else 0), _ptr(tc_status(qkv.device)), _stream())
 
 
 def attention_prefill_tcgen05_wait_probe(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads: int, scale: float,
