@@ -26,7 +26,9 @@ and gated linear attention, a routed feed-forward) beside Datasun and Qwen3, wit
 of every kernel of a prompt step and of a single-token step.  ``--design munerax`` and
 ``--design kikelorn`` do it for those designs (Kikelorn: chunked attention, latent attention with a
 query latent, a minGRU and chunked attention again, in out-norm blocks) beside the designs closest
-to them and Qwen3.
+to them and Qwen3, and ``--design zirivik`` for Zirivik (two retention layers, an attention layer with a
+window and kept first tokens, and one that reads its keys; dense and routed feed-forwards in turn)
+beside Bepilorn, Datasun and Qwen3.
 
 The work is one GPU's: for ``--gpus`` above 1 it says so and exits with 2.  The reference arm
 (``--impl reference``) is unavailable: the reference is a Rust workspace, there is no Rust
@@ -403,6 +405,27 @@ def kikelorn_config(width, heads, kv, d, ff, layers):
             "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
 
 
+ZIRIVIK_KEEP = 4               # first tokens the windowed layers keep in the design runs
+
+
+def zirivik_config(width, heads, kv, d, ff, layers):
+    """A Zirivik model of these layer sizes: of every four layers two are retention (heads of the
+    attention's sizes, whole-head rotation, decays as Datasun's in these runs), the third is attention
+    over a window and the first four tokens, the fourth the same with the third's keys and values; dense
+    feed-forwards in even layers, routed ones in odd layers whose four used experts together have the
+    dense inner size."""
+    ret = {"heads": heads, "dim": d, "vdim": d, "rot": {"base": 1e6, "dims": d},
+           "decay": [1.0 - 2.0 ** -(5.0 + 3.0 * i / max(heads - 1, 1)) for i in range(heads)]}
+    att = {"heads": heads, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": DESIGN_WINDOW, "keep_first": ZIRIVIK_KEEP}}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4, "limit": 7.0}, "router": {"experts": BEPILORN_EXPERTS, "top": 4}}
+    out = []
+    for i in range(layers):
+        mixer = ret if i % 4 < 2 else (att if i % 4 == 2 else dict(att, kv_from=i - 1))
+        out.append({"type": "retention" if i % 4 < 2 else "attention", "mixer": mixer, "mlp": moe if i % 2 else {"kind": "dense", "ff": ff}})
+    return {"architecture": "Zirivik", "vocab": DESIGN_VOCAB, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "logit_softcap": 30.0, "layers": out}
+
+
 def decode_breakdown(model, batch, ctx_len):
     """One instrumented single-token step (no graph, an event around every kernel) behind prompts of
     ``ctx_len`` tokens: milliseconds by kernel."""
@@ -436,12 +459,14 @@ def design_run(a) -> int:
         width, heads, kv, d, ff = DESIGN_SIZES[name]
         qwen3 = dict(CONFIG_4B, num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads,
                      num_key_value_heads=kv, head_dim=d, intermediate_size=ff, vocab_size=DESIGN_VOCAB)
-        if a.design == "kikelorn":      # beside the design with the same latent attention, the one with chunked attention and a recurrence, and the dense one
+        if a.design == "zirivik":       # beside the design with the same block and a routed feed-forward, the one with the same recurrence and windows, and the dense one
+            configs = {"zirivik": zirivik_config(width, heads, kv, d, ff, layers),
+                       "bepilorn": bepilorn_config(width, heads, kv, d, ff, layers),
+                       "datasun": datasun_config(width, heads, kv, d, ff, layers), "qwen3": qwen3}
+        elif a.design == "kikelorn":    # beside the design with the same latent attention, the one with chunked attention and a recurrence, and the dense one
             configs = {"kikelorn": kikelorn_config(width, heads, kv, d, ff, layers),
                        "munerax": munerax_config(width, heads, kv, d, ff, layers),
                        "bepilorn": bepilorn_config(width, heads, kv, d, ff, layers), "qwen3": qwen3}
-            if a.only:
-                configs = {k: v for k, v in configs.items() if k in a.only.split(",")}
         elif a.design == "munerax":     # beside the routed design and beside the dense softmax-attention one
             configs = {"munerax": munerax_config(width, heads, kv, d, ff, layers),
                        "bepilorn": bepilorn_config(width, heads, kv, d, ff, layers), "qwen3": qwen3}
@@ -450,9 +475,11 @@ def design_run(a) -> int:
                        "datasun": datasun_config(width, heads, kv, d, ff, layers), "qwen3": qwen3}
         else:
             configs = {"datasun": datasun_config(width, heads, kv, d, ff, layers), "qwen3": qwen3}
+        if a.only:
+            configs = {k: v for k, v in configs.items() if k in a.only.split(",")}
         for design, cfg in configs.items():
             model = Model.from_random(cfg, seed=0, dtype="bfloat16", max_tokens=64 * 2048, max_seq_len=CONTEXT, max_batch=64)
-            by_kernel = a.design in ("bepilorn", "munerax", "kikelorn")
+            by_kernel = a.design in ("bepilorn", "munerax", "kikelorn", "zirivik")
             pf = prefill_run(model, PREFILL_TOKENS, 5, layers, breakdown=True, by_kernel=by_kernel)
             row = {"prefill_2048": {"ms": round(pf["ms"], 3), "tok_s": round(pf["tok_s"], 1), "breakdown": pf["breakdown"]}}
             for b in (8, 64):
@@ -472,9 +499,11 @@ def design_run(a) -> int:
                           "layer 0, then %d experts, 4 used, and a shared one" % (MUNERAX_LATENT, BEPILORN_EXPERTS),
                "kikelorn": "chunked attention (chunk %d, %d taps on q, k, v), latent attention (cache row %d + head/2, query latent), "
                            "minGRU, chunked attention; out-norm blocks with %d taps in front of every sublayer and a gate behind it; "
-                           "dense feed-forward with biases" % (DESIGN_WINDOW, KIKELORN_TAPS, MUNERAX_LATENT, KIKELORN_TAPS)}[a.design]
+                           "dense feed-forward with biases" % (DESIGN_WINDOW, KIKELORN_TAPS, MUNERAX_LATENT, KIKELORN_TAPS),
+               "zirivik": "retention x2, attention (window %d and the first %d tokens) x1 and one that reads its keys; dense feed-forward "
+                          "in even layers, %d experts, 4 used, in odd ones" % (DESIGN_WINDOW, ZIRIVIK_KEEP, BEPILORN_EXPERTS)}[a.design]
     beside = {"bepilorn": "datasun and qwen3", "munerax": "bepilorn and qwen3",
-              "kikelorn": "munerax, bepilorn and qwen3"}.get(a.design, "qwen3")
+              "kikelorn": "munerax, bepilorn and qwen3", "zirivik": "bepilorn, datasun and qwen3"}.get(a.design, "qwen3")
     print(json.dumps({"workloads": a.design + " beside " + beside
                       + " at equal layer sizes, builder-run beside the benchmark", "dtype": "bf16",
                       "layers": layers, "pattern": pattern, "vocab": DESIGN_VOCAB,
@@ -490,7 +519,8 @@ def kernel_run(a) -> int:
     """Times ONE kernel on one workload (for profiling under ncu and for the files in profiles/):
     ``--kernel skinny_gemm|gemm_tcgen05 --shape qkv|o|gateup|down|head --rows M`` or
     ``--kernel attention_decode|attention_prefill|attention_prefill_tcgen05 --rows B_or_T --ctx C``
-    (``--seqs N``: N prompts of --rows tokens each),
+    (``--seqs N``: N prompts of --rows tokens each; ``--window W --keep-first K --exact-weights``: the masked and exact forms),
+    ``--kernel lightning_chunks --seqs N --rows T`` / ``--kernel lightning_scan --rows B`` (``--rotate``: as retention),
     ``--kernel qk_norm_rope --rows T``, ``--kernel decay_scan --rows T [--seqs N]`` / ``--kernel decay_step --rows B`` (the
     recurrence with a step size per head over prompts / over single tokens), ``--kernel attention_latent --seqs N --rows T --ctx C
     --heads H`` (the latent attention; --rows 1: single tokens behind C cached ones), ``--kernel weight_stream --shape S [--stages R] [--ksplit Z]`` (the
@@ -547,18 +577,24 @@ def kernel_run(a) -> int:
         decay = torch.linspace(0.96, 0.996, h, device=dev, dtype=torch.float32)
         cu = torch.arange(0, (n_seq + 1) * t_new, t_new, dtype=torch.int32, device=dev)
         slots = torch.arange(n_seq, dtype=torch.int32, device=dev)
+        kw = {"act": ops.LIGHT_ACT_SILU}
+        if a.rotate:
+            from builderforce_inference_b200.parts.rotary import rotary_table
+            pos = torch.arange(t_new, dtype=torch.int32, device=dev).repeat(n_seq)
+            kw = {"act": ops.LIGHT_ACT_NONE, "rope_table": rotary_table(1e6, d, max(t_new, 2), dev), "rot_dim": d, "token_pos": pos,
+                  "k_scale": d ** -0.5}
 
         def one(i):
             if chunks:
-                if not fast_ops.lightning_chunks_bf16(proj, 0, h * d, 2 * h * d, o, states[0], decay, cu, slots, n_seq, h, d, d):
+                if not fast_ops.lightning_chunks_bf16(proj, 0, h * d, 2 * h * d, o, states[0], decay, cu, slots, n_seq, h, d, d, **kw):
                     raise SystemExit("lightning_chunks does not take this shape")
             else:
                 ops.lightning_scan(proj, 0, h * d, 2 * h * d, o, states[i % copies], decay, cu, slots, n_seq, h, d, d,
-                                   ops.LIGHT_ACT_SILU, True, True)
+                                   few_tokens=True, single_tokens=True, **kw)
         bytes_moved = n_seq * h * d * d * 4 * 2 + n_seq * t_new * (3 * h * d * 2 + h * d * 4)
         # per token and head: scores and their use within a chunk (causal half of 64 x 64), q S and the state update
         flops = n_seq * t_new * h * (2.0 * d * d * 2 + (2.0 * 32 * (d + d) if chunks else 0.0))
-        what = {"seqs": n_seq, "new_tokens": t_new, "heads": h, "dim": d, "vdim": d}
+        what = {"seqs": n_seq, "new_tokens": t_new, "heads": h, "dim": d, "vdim": d, "rotate": bool(a.rotate)}
     elif a.kernel in ("causal_conv", "gated_scan", "norm_add_gated", "bias_gelu"):
         # the kernels around an out-norm block's sublayers and of the minGRU: --seqs prompts of --rows tokens, --width channels
         from builderforce_inference_b200.kernels import ops
@@ -745,7 +781,8 @@ def kernel_run(a) -> int:
         cache_bytes = n_pages * nkv * 64 * d * 2 * 2
         copies = max(2, int(400e6 // cache_bytes) + 1) if decode else 1
         kvs = [KVView(torch.randn(n_pages, nkv, 64, d, device=dev, dtype=torch.bfloat16),
-                      torch.randn(n_pages, nkv, 64, d, device=dev, dtype=torch.bfloat16), table, nkv, d, None)
+                      torch.randn(n_pages, nkv, 64, d, device=dev, dtype=torch.bfloat16), table, nkv, d,
+                      a.window or None, keep_first=a.keep_first)
                for _ in range(copies)]
         q = torch.randn(n_seq * t_new, (nq + 2 * nkv) * d, device=dev, dtype=torch.bfloat16)
         out = torch.empty(n_seq * t_new, nq * d, device=dev, dtype=torch.bfloat16)
@@ -763,11 +800,18 @@ def kernel_run(a) -> int:
         fn = {"attention_decode": fast_ops.attention_decode_bf16, "attention_prefill": fast_ops.attention_prefill_bf16,
               "attention_prefill_tcgen05": fast_ops.attention_prefill_tcgen05_bf16}[a.kernel]
         def one(i):
-            if not fn(ctx, q, out, kvs[i % copies], nq, d ** -0.5):
+            if not fn(ctx, q, out, kvs[i % copies], nq, d ** -0.5, exact_weights=a.exact_weights):
                 raise SystemExit(f"{a.kernel} does not take this shape")
-        bytes_moved = n_seq * ctx_len * 2 * nkv * d * 2
-        flops = 4.0 * nq * d * n_seq * (ctx_len if decode else t_new * (t_new + 1) / 2)
-        what = {"seqs": n_seq, "new_tokens": t_new, "context": ctx_len, "q_heads": nq, "kv_heads": nkv, "head_dim": d}
+
+        def visible(pos):               # keys the token at pos reads
+            lo = max(0, pos - a.window + 1) if a.window else 0
+            return pos + 1 - lo + min(a.keep_first, lo)
+        bytes_moved = n_seq * (visible(ctx_len - 1) if decode else ctx_len) * 2 * nkv * d * 2
+        if not decode:
+            bytes_moved += n_seq * t_new * nq * d * 2 * 2          # q in, the heads' outputs out
+        flops = 4.0 * nq * d * n_seq * sum(visible(p) for p in range(ctx_len - t_new, ctx_len))
+        what = {"seqs": n_seq, "new_tokens": t_new, "context": ctx_len, "q_heads": nq, "kv_heads": nkv, "head_dim": d,
+                "window": a.window, "keep_first": a.keep_first, "exact_weights": bool(a.exact_weights)}
     for i in range(3):
         one(i)
     torch.cuda.synchronize()
@@ -919,10 +963,14 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=None, help="run fewer layers of the same sizes")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 points and the prefill")
-    ap.add_argument("--design", default=None, choices=["datasun", "bepilorn", "munerax", "kikelorn"],
+    ap.add_argument("--design", default=None, choices=["datasun", "bepilorn", "munerax", "kikelorn", "zirivik"],
                     help="instead of the benchmark: this design beside qwen3 at equal layer sizes (see design_run)")
     ap.add_argument("--sizes", default=None, help="with --design: names of DESIGN_SIZES, comma-separated (default: all)")
-    ap.add_argument("--only", default=None, help="with --design kikelorn: the designs to run, comma-separated (default: all four)")
+    ap.add_argument("--only", default=None, help="with --design: the designs to run, comma-separated (default: all of that run)")
+    ap.add_argument("--window", type=int, default=0, help="kernel mode, attention: the last --window positions")
+    ap.add_argument("--keep-first", type=int, default=0, help="kernel mode, attention: and the first --keep-first positions")
+    ap.add_argument("--exact-weights", action="store_true", help="kernel mode, attention: weights float32 in effect")
+    ap.add_argument("--rotate", action="store_true", help="kernel mode, lightning: retention (rotated q and k, no activations)")
     a = ap.parse_args()
     if a.impl == "reference":
         print(json.dumps({"impl": "reference", "unavailable":

@@ -951,6 +951,95 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ x, long x_stri
     }
 }
 
+// The same for parts of a multiple of 4 values up to 32 * 4 * VPL: a lane keeps its share of a part (16-byte pieces)
+// in registers, so everything is read once.
+__device__ __forceinline__ float4 rec_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 rec_load4(const bf16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+    const float2 a = __bfloat1622float2(h2[0]), b = __bfloat1622float2(h2[1]);
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void rec_store4(float* p, const float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void rec_store4(bf16* p, const float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 packed;
+    packed.x = *reinterpret_cast<const uint32_t*>(&lo);
+    packed.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = packed;
+}
+
+template <typename T, int VPL>
+__global__ void __launch_bounds__(256)
+gated_group_norm_vec_kernel(const float* __restrict__ x, long x_stride, const T* __restrict__ gate, long gate_stride,
+                            const void* __restrict__ w, int w_dtype, int w_len, T* __restrict__ y, long y_stride, int width,
+                            int parts, int gate_first, int gate_act, float eps) {
+    pdl_trigger();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    const int t = blockIdx.x, p = blockIdx.y * n_warps + warp;
+    const int len = width / parts, n4 = len >> 2, j0 = p * len;
+    pdl_wait();
+    if (p >= parts) return;
+    const float* xr = x + (size_t)t * x_stride + j0;
+    const T* gr = gate + (size_t)t * gate_stride + j0;
+    T* yr = y + (size_t)t * y_stride + j0;
+    float4 v[VPL], g[VPL];
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) {
+        const int j = i * 32 + lane;
+        v[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < n4) v[i] = rec_load4(xr + j * 4), g[i] = rec_load4(gr + j * 4);
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) {
+        float4& a = g[i];
+        if (gate_act) a = make_float4(rec_silu(a.x), rec_silu(a.y), rec_silu(a.z), rec_silu(a.w));
+        else a = make_float4(rec_sigmoid(a.x), rec_sigmoid(a.y), rec_sigmoid(a.z), rec_sigmoid(a.w));
+        if (gate_first) {
+            const float4 u = make_float4(v[i].x * a.x, v[i].y * a.y, v[i].z * a.z, v[i].w * a.w);
+            ss = fmaf(u.x, u.x, ss), ss = fmaf(u.y, u.y, ss), ss = fmaf(u.z, u.z, ss), ss = fmaf(u.w, u.w, ss);
+        } else {
+            ss = fmaf(v[i].x, v[i].x, ss), ss = fmaf(v[i].y, v[i].y, ss), ss = fmaf(v[i].z, v[i].z, ss), ss = fmaf(v[i].w, v[i].w, ss);
+        }
+    }
+    ss = warp_sum(ss);
+    const float scale = 1.0f / sqrtf(ss / (float)len + eps);
+#pragma unroll
+    for (int i = 0; i < VPL; ++i) {
+        const int j = i * 32 + lane;
+        if (j >= n4) continue;
+        float4 o = make_float4(v[i].x * g[i].x * scale, v[i].y * g[i].y * scale, v[i].z * g[i].z * scale, v[i].w * g[i].w * scale);
+        if (w != nullptr) {
+            const int c = (j0 + j * 4) % w_len;             // w_len is a multiple of 4
+            o.x *= load_as_f32(w, w_dtype, c), o.y *= load_as_f32(w, w_dtype, c + 1);
+            o.z *= load_as_f32(w, w_dtype, c + 2), o.w *= load_as_f32(w, w_dtype, c + 3);
+        }
+        rec_store4(yr + j * 4, o);
+    }
+}
+
+template <typename T>
+static bool launch_group_norm_vec(const float* x, long x_stride, const T* gate, long gate_stride, const void* w, int w_dtype,
+                                  int w_len, T* y, long y_stride, int n_rows, int width, int parts, int gate_first, int gate_act,
+                                  float eps, cudaStream_t stream) {
+    const int len = width / parts, piece = 4 * (int)sizeof(T);
+    const auto al = [](const void* p, int n) { return ((uintptr_t)p & (uintptr_t)(n - 1)) == 0; };
+    if (width < 512 || len % 4 != 0 || len > 512 || x_stride % 4 != 0 || gate_stride % 4 != 0 || y_stride % 4 != 0 || !al(x, 16) || !al(gate, piece) ||
+        !al(y, piece) || (w != nullptr && w_len % 4 != 0))
+        return false;
+    const int warps = parts < 8 ? parts : 8;
+    const dim3 grid(n_rows, (parts + warps - 1) / warps), block(32 * warps);
+#define BFI_GROUP_NORM(V)                                                                                                   \
+    bfi_launch(gated_group_norm_vec_kernel<T, V>, grid, block, 0, stream, x, x_stride, gate, gate_stride, w, w_dtype, w_len, \
+               y, y_stride, width, parts, gate_first, gate_act, eps)
+    if (len <= 128) BFI_GROUP_NORM(1);
+    else if (len <= 256) BFI_GROUP_NORM(2);
+    else BFI_GROUP_NORM(4);
+#undef BFI_GROUP_NORM
+    return true;
+}
+
 extern "C" int bfi_gated_group_norm(const float* x, long x_stride, const void* gate, long gate_stride, int dtype,
                                     const void* w, int w_dtype, int w_len, void* y, long y_stride, int n_rows, int width,
                                     int parts, int gate_first, int gate_act, float eps, cudaStream_t stream) {
@@ -960,6 +1049,11 @@ extern "C" int bfi_gated_group_norm(const float* x, long x_stride, const void* g
     BFI_REQUIRE(w_len > 0 && width % w_len == 0, "gated_group_norm: a weight of %d values does not repeat along %d", w_len, width);
     BFI_REQUIRE(x_stride >= width && gate_stride >= width && y_stride >= width, "gated_group_norm: row stride shorter than the row");
     if (n_rows == 0) return 0;
+    if (dtype == BFI_F32 ? launch_group_norm_vec<float>(x, x_stride, (const float*)gate, gate_stride, w, w_dtype, w_len, (float*)y, y_stride,
+                                                        n_rows, width, parts, gate_first, gate_act, eps, stream)
+                         : launch_group_norm_vec<bf16>(x, x_stride, (const bf16*)gate, gate_stride, w, w_dtype, w_len, (bf16*)y, y_stride,
+                                                       n_rows, width, parts, gate_first, gate_act, eps, stream))
+        return bfi_check_launch("gated_group_norm");
     int warps = parts < 8 ? parts : 8;
     if (dtype == BFI_F32)
         bfi_launch(gated_group_norm_kernel<float>, dim3(n_rows), dim3(32 * warps), 0, stream, x, x_stride, (const float*)gate,

@@ -153,12 +153,13 @@ norm_add_vec_kernel(float* __restrict__ x, long x_stride, const float* __restric
     const int t = blockIdx.x;
     const int n4 = width >> 2;
     // the weights and the gate's bias do not come from the kernel before this one: fetched before the wait
-    float4 wv[EARLY ? VPT : 1];
+    float4 wv[EARLY ? VPT : 1], wv2[EARLY ? VPT : 1];
     if (EARLY) {
 #pragma unroll
         for (int i = 0; i < VPT; ++i) {
             const int j = i * 256 + threadIdx.x;
             wv[i] = j < n4 ? load4_as_f32(w, w_dtype, (size_t)j * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+            wv2[i] = j < n4 && h != nullptr ? load4_as_f32(w2, w2_dtype, (size_t)j * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
     pdl_wait();
@@ -236,12 +237,9 @@ norm_add_vec_kernel(float* __restrict__ x, long x_stride, const float* __restric
     for (int i = 0; i < VPT; ++i) {
         const int j = i * 256 + threadIdx.x;
         if (j >= n4) continue;
-        const int c = j * 4;
-        const size_t at = (size_t)t * h_stride + c;
-        store_from_f32(h, h_dtype, at, v[i].x * scale2 * load_as_f32(w2, w2_dtype, c));
-        store_from_f32(h, h_dtype, at + 1, v[i].y * scale2 * load_as_f32(w2, w2_dtype, c + 1));
-        store_from_f32(h, h_dtype, at + 2, v[i].z * scale2 * load_as_f32(w2, w2_dtype, c + 2));
-        store_from_f32(h, h_dtype, at + 3, v[i].w * scale2 * load_as_f32(w2, w2_dtype, c + 3));
+        const float4 ww = EARLY ? wv2[i] : load4_as_f32(w2, w2_dtype, (size_t)j * 4);
+        store4_from_f32(h, h_dtype, (size_t)t * h_stride + j * 4,
+                        make_float4(v[i].x * scale2 * ww.x, v[i].y * scale2 * ww.y, v[i].z * scale2 * ww.z, v[i].w * scale2 * ww.w));
     }
 }
 
@@ -272,14 +270,15 @@ extern "C" int bfi_norm_add(float* x, long x_stride, const float* y, long y_stri
     g.logits = gate, g.dtype = gate_dtype, g.stride = gate_stride, g.bias = gate != nullptr ? gate_bias : nullptr;
     g.bias_dtype = gate_bias_dtype;
     const auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    // the plain normed add keeps the kernel (and with it the order of its sums) it has always had
     const auto al_for = [](const void* p, int dt) { return (reinterpret_cast<uintptr_t>(p) & (dt == BFI_F32 ? 15 : 7)) == 0; };
     const auto al_out = [](const void* p, long stride, int dt) {
         return (reinterpret_cast<uintptr_t>(p) & (dt == BFI_F32 ? 15 : 7)) == 0 && stride % 4 == 0;
     };
     const bool tail_ok = conv_w == nullptr || (al_out(conv_h, conv_h_stride, conv_out_dtype) && al_out(conv_plain, conv_plain_stride, conv_out_dtype) &&
                                                (reinterpret_cast<uintptr_t>(conv_state) & 15) == 0);
-    if ((gate != nullptr || mult != 1.0f || conv_w != nullptr) && tail_ok && al_for(w, w_dtype) && (gate_bias == nullptr || al_for(gate_bias, gate_bias_dtype)) && width % 4 == 0 &&
+    const bool next_ok = h == nullptr || (al_out(h, h_stride, h_dtype) && al_for(w2, w2_dtype));
+    // short rows have no use for it: they keep the plain kernel
+    if ((gate != nullptr || mult != 1.0f || conv_w != nullptr || width >= 512) && tail_ok && next_ok && al_for(w, w_dtype) && (gate_bias == nullptr || al_for(gate_bias, gate_bias_dtype)) && width % 4 == 0 &&
         width <= 8 * 4 * 256 && x_stride % 4 == 0 && y_stride % 4 == 0 && al16(x) && al16(y) &&
         (gate == nullptr || (gate_stride % 4 == 0 && (((uintptr_t)gate) & (gate_dtype == BFI_F32 ? 15 : 7)) == 0))) {
         const int vpt = (width / 4 + 255) / 256;

@@ -169,7 +169,7 @@ def random_config(seed):
         if kind == "retention":
             h, d = rng.choice([1, 2, 3, 4]), rng.choice([4, 8, 16, 24, 32, 64, 128])
             rot = (rng.choice([100.0, 1e4, 1e6]), rng.choice(list(range(2, d + 1, 2)) + [d] * 3)) if rng.random() < 0.85 else None
-            lay = ret(d, rng.choice([1, 4, 8, 16, 32, 48, 64, d]), [rng.choice([0.0, 0.5, 0.9, 0.97, 0.99, 0.999, 1.0]) for _ in range(h)], rot)
+            lay = ret(d, rng.choice([16 // h + 1, 8 + 4 * (h < 2), 16, 32, 48, 64, max(d, 16 // h + 1)]), [rng.choice([0.0, 0.5, 0.9, 0.97, 0.99, 0.999, 1.0]) for _ in range(h)], rot)
         else:
             if lenders and rng.random() < 0.45:
                 src = rng.choice(lenders)
@@ -178,17 +178,17 @@ def random_config(seed):
             else:
                 src = None
                 g = rng.choice([1, 2, 3])
-                a, d, dv = g * rng.choice([1, 2, 4]), rng.choice([2, 8, 16, 32, 48, 64, 128]), rng.choice([1, 8, 16, 40, 64])
-                if rng.random() < 0.4:
+                a, d, dv = g * rng.choice([1, 2, 4]), rng.choice([2, 8, 16, 32, 48, 64, 128]), rng.choice([16 // g, 16, 24, 40, 64])
+                if rng.random() < 0.4 and g * d >= 16:
                     dv = d
                 lenders.append(i)
             lay = att(a, g, d, dv, rng.choice([0.1, d ** -0.5, 0.4]), *mask(), kv_from=src)
         mlp = rng.choice([None, "dense", "moe", "moe"])
         if mlp == "dense":
-            mlp = dense(rng.choice([1, 20, 64, 100]))
+            mlp = dense(rng.choice([16, 20, 64, 100]))
         elif mlp == "moe":
             e = rng.choice([1, 2, 5, 8, 16])
-            mlp = moe(e, rng.randint(1, min(e, 4)), rng.choice([4, 20, 32, 64]), rng.choice([0.2, 1.0, 7.0]))
+            mlp = moe(e, rng.randint(1, min(e, 4)), rng.choice([12, 20, 32, 64]), rng.choice([0.2, 1.0, 7.0]))
         layers.append((lay, mlp))
     cfg = config(rng.choice([97, 256, 333]), width, rng.choice([1e-6, 1e-5]), rng.choice([1.0, 0.5, math.sqrt(width)]),
                  rng.choice([5.0, 30.0]), layers)
