@@ -174,7 +174,8 @@ struct FtItem {
     int n_keep;       // tiles of kept first positions at the head of the list: tile i is i for i < n_keep, else j_beg + i - n_keep
 };
 
-template <int D, bool SPLIT_P>
+// KEEP: there may be kept first positions (without them the kernel is the one for plain windows).
+template <int D, bool SPLIT_P, bool KEEP>
 __global__ void __launch_bounds__(FT_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, long out_stride,
@@ -297,9 +298,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 const int hi_block = p.start + min(p.tok0 + FT_ROWS - 1, p.nt - 1);
                 const int lo_block = window > 0 ? max(0, p0 - window + 1) : 0;
                 p.j_beg = lo_block / FT_KEYS;
-                p.n_keep = min((keep_first + FT_KEYS - 1) / FT_KEYS, p.j_beg);
+                p.n_keep = KEEP ? min((keep_first + FT_KEYS - 1) / FT_KEYS, p.j_beg) : 0;
                 p.n_tiles = p.n_keep + hi_block / FT_KEYS - p.j_beg + 1;               // key tiles
-                const int j0 = p.n_keep > 0 ? 0 : p.j_beg;
+                const int j0 = KEEP && p.n_keep > 0 ? 0 : p.j_beg;
                 p.pg0 = page_of(p.slot, 2 * j0);
                 p.pg1 = page_of(p.slot, 2 * j0 + 1);
                 return p;
@@ -323,7 +324,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     items[qi].row0 = p.t0 + p.tok0;
                     items[qi].rows = p.nt - p.tok0;
                     items[qi].head = p.head;
-                    items[qi].n_keep = p.n_keep;
+                    if (KEEP) items[qi].n_keep = p.n_keep;
                     mbar_expect_tx(&q_full[qi], TILE_BYTES);
                     for (int c = 0; c < BOXES; ++c)
                         tma_load_2d(q_smem + (size_t)qi * TILE_BYTES + c * FT_BOX_BYTES, &map_q, p.head * D + c * 64,
@@ -338,7 +339,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         bool failed = !announce(0, cur);
         for (int it = 0; !failed && cur.have; ++it, cur = nxt) {
             int ok = 1;
-            const int kvh = cur.kvh, slot = cur.slot, j_beg = cur.j_beg, n_keep = cur.n_keep, n_tiles = cur.n_tiles;
+            const int kvh = cur.kvh, slot = cur.slot, j_beg = cur.j_beg, n_keep = KEEP ? cur.n_keep : 0, n_tiles = cur.n_tiles;
             const int seq_hi = cur.start + cur.nt - 1;                          // last position the cache holds
             int pg_next[2] = {cur.pg0, cur.pg1};
             for (int i = 0; i < n_tiles; ++i, ++g) {
@@ -520,7 +521,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             const int qi = it & 1;
             if (!__all_sync(FULL, MBAR_WAIT(&q_full[qi], (uint32_t)(it >> 1) & 1))) { ok = false; timed_out = true; break; }
             const int n_tiles = items[qi].n_tiles, j_beg = items[qi].j_beg, p0 = items[qi].p0, seq_hi = items[qi].seq_hi;
-            const int row0 = items[qi].row0, rows = items[qi].rows, head = items[qi].head, n_keep = items[qi].n_keep;
+            const int row0 = items[qi].row0, rows = items[qi].rows, head = items[qi].head, n_keep = KEEP ? items[qi].n_keep : 0;
             __syncwarp();
             if (lane == 0) mbar_arrive(&q_empty[qi]);
             if (n_tiles == 0) break;
@@ -548,9 +549,9 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     const int hi = pos_r - key0, lo = lo_r - key0, keep = keep_first - key0;     // ... or index < keep
 #pragma unroll
                     for (int c = 0; c < FT_KEYS / 32; ++c) {
-                        if (__all_sync(FULL, c * 32 + 31 <= hi && (c * 32 >= lo || c * 32 + 31 < keep))) continue;
+                        if (__all_sync(FULL, c * 32 + 31 <= hi && (c * 32 >= lo || (KEEP && c * 32 + 31 < keep)))) continue;
 #pragma unroll
-                        for (int e = c * 32; e < c * 32 + 32; ++e) s[e] = (e > hi || (e < lo && e >= keep)) ? -INFINITY : s[e];
+                        for (int e = c * 32; e < c * 32 + 32; ++e) s[e] = (e > hi || (e < lo && (!KEEP || e >= keep))) ? -INFINITY : s[e];
                     }
                 }
                 float mx = s[0];
@@ -663,7 +664,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     BFI_TRACE_END();
 }
 
-template <int D, bool SPLIT_P>
+template <int D, bool SPLIT_P, bool KEEP>
 static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out_stride, const void* k_pages,
                              const void* v_pages, long n_pages, const int* block_table, int table_stride,
                              const int* cu_seqlens, const int* seq_slot, const int* seq_start, int n_seqs, long n_tokens,
@@ -680,7 +681,7 @@ static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out
     // at least half an SM's shared memory, so that two blocks never share one SM's tensor memory
     const size_t tiles = (size_t)6 * TILE_BYTES + 1024 + 512 + FT_META_SEQS * sizeof(int4) + 4 * 4096;
     const size_t smem = tiles > 120 * 1024 ? tiles : 120 * 1024;
-    auto kernel = attention_prefill_tc_kernel<D, SPLIT_P>;
+    auto kernel = attention_prefill_tc_kernel<D, SPLIT_P, KEEP>;
     static bool configured = false;
     const int n_sm = bfi_sm_count();
     if (!configured) {
@@ -723,14 +724,20 @@ static int attention_prefill_tc_launch(const void* qkv, long q_stride, void* out
         ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15) || (long)((max_seq_tokens + FT_ROWS - 1) / FT_ROWS) * n_seqs * n_q > 0x3fffffffL)
         return 2;
     if (n_pages * n_kv * FT_PAGE > 0x7fffffffL) return 2;       // TMA coordinates are 32-bit
-#define BFI_PREFILL_TC(DD, SP)                                                                                              \
-    return launch_prefill_tc<DD, SP>(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,   \
+#define BFI_PREFILL_TC(DD, SP, KP)                                                                                              \
+    return launch_prefill_tc<DD, SP, KP>(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,   \
                                      cu_seqlens, seq_slot, seq_start, n_seqs, n_tokens, max_seq_tokens, n_q, n_kv, window,   \
                                      keep_first, scale, sink, status, stream, waits)
-    if (d == 64 && split_p) BFI_PREFILL_TC(64, true);
-    if (d == 64) BFI_PREFILL_TC(64, false);
-    if (split_p) BFI_PREFILL_TC(128, true);
-    BFI_PREFILL_TC(128, false);
+    if (split_p) {
+        if (d == 64) BFI_PREFILL_TC(64, true, true);
+        BFI_PREFILL_TC(128, true, true);
+    }
+    if (keep_first > 0) {
+        if (d == 64) BFI_PREFILL_TC(64, false, true);
+        BFI_PREFILL_TC(128, false, true);
+    }
+    if (d == 64) BFI_PREFILL_TC(64, false, false);
+    BFI_PREFILL_TC(128, false, false);
 #undef BFI_PREFILL_TC
 }
 

@@ -51,8 +51,10 @@ struct TcConfig {
 
 // ------------------------------------------------------------------------------------------
 // The kernel.  grid = (row tiles of W, token tiles, splits of K)
+// MAPPED (here and in the many-row kernel): the epilogue does something to the accumulators before the
+// epilogues the other instantiations have: the squared ReLU, or factors on the gated product's input.
 // ------------------------------------------------------------------------------------------
-template <int BT>
+template <int BT, bool MAPPED>
 __global__ void __launch_bounds__(TC_THREADS, TcConfig<BT>::BLOCKS_PER_SM)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
                     void* __restrict__ C, int c_dtype, long ldc, int M, int N, int K, int kblocks_per_split,
@@ -208,7 +210,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                 float v[16];
                 tmem_ld16(lane_addr + c * 16, v);
                 if (epilogue == EPI_SWIGLU) {
-                    if (gate.in_scale != nullptr) {
+                    if (MAPPED && gate.in_scale != nullptr) {
 #pragma unroll
                         for (int j = 0; j < 16; ++j)
                             v[j] *= (j < rows_here && n < N) ? gate_in_scale(gate, m_c + j, n >> 1) : 0.0f;
@@ -230,7 +232,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         for (int j = 0; j < 16; ++j)
                             if (j < rows_here) c_io[(size_t)j * ldc] = old[j] + v[j];
                     } else {
-                        if (epilogue == BFI_EPI_RELU_SQUARED) {
+                        if (MAPPED && epilogue == BFI_EPI_RELU_SQUARED) {
 #pragma unroll
                             for (int j = 0; j < 16; ++j) v[j] = relu_squared(v[j]);
                         }
@@ -291,7 +293,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
 #pragma unroll
                     for (int r = 0; r < 8; ++r) v += x[u][r];
                     if (epilogue == EPI_SWIGLU) {
-                        if (gate.in_scale != nullptr) v *= (live && n < N) ? gate_in_scale(gate, m, n >> 1) : 0.0f;
+                        if (MAPPED && gate.in_scale != nullptr) v *= (live && n < N) ? gate_in_scale(gate, m, n >> 1) : 0.0f;
                         const float act = gate_mul_fast(v, __shfl_down_sync(0xffffffffu, v, 1), gate);
                         if (live && (lane & 1) == 0 && n + 1 < N) store_from_f32(C, c_dtype, (size_t)m * ldc + (n >> 1), act);
                     } else if (live && n < N) {
@@ -299,7 +301,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                         if (epilogue == EPI_ACCUMULATE)
                             reinterpret_cast<float*>(C)[o] = old[u] + v;
                         else
-                            store_from_f32(C, c_dtype, o, epilogue == BFI_EPI_RELU_SQUARED ? relu_squared(v) : v);
+                            store_from_f32(C, c_dtype, o, MAPPED && epilogue == BFI_EPI_RELU_SQUARED ? relu_squared(v) : v);
                     }
                 }
             }
@@ -471,7 +473,7 @@ __device__ __forceinline__ void tp_pre_store(float (&v)[16], int epilogue, const
     }
 }
 
-template <int HALVES>
+template <int HALVES, bool MAPPED>
 __global__ void __launch_bounds__(TP_THREADS, 1)
 gemm_tcgen05_prefill_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                             void* __restrict__ C, int c_dtype, long ldc, int M, int N, int K, int tiles_m, int tiles_n,
@@ -668,14 +670,14 @@ gemm_tcgen05_prefill_kernel(const __grid_constant__ CUtensorMap map_a, const __g
                         float v[4][16];
                         tmem_ld64(taddr + c_direct * 16, v);
 #pragma unroll
-                        for (int g = 0; g < 4; ++g) tp_pre_store(v[g], epilogue, gate, m, n0 + g * 16, M, N);
+                        for (int g = 0; g < (MAPPED ? 4 : 0); ++g) tp_pre_store(v[g], epilogue, gate, m, n0 + g * 16, M, N);
                         tp_emit_group<4>(stage, v, lane, epilogue, gate, c_dtype, C, ldc, m_base, M, n0);
                         c_direct += 4;
                     } else if (c_direct + 2 <= c_end && n0 + 32 <= N) {
                         float v[2][16];
                         tmem_ld32(taddr + c_direct * 16, v);
 #pragma unroll
-                        for (int g = 0; g < 2; ++g) tp_pre_store(v[g], epilogue, gate, m, n0 + g * 16, M, N);
+                        for (int g = 0; g < (MAPPED ? 2 : 0); ++g) tp_pre_store(v[g], epilogue, gate, m, n0 + g * 16, M, N);
                         tp_emit_group<2>(stage, v, lane, epilogue, gate, c_dtype, C, ldc, m_base, M, n0);
                         c_direct += 2;
                     } else {
@@ -690,7 +692,7 @@ gemm_tcgen05_prefill_kernel(const __grid_constant__ CUtensorMap map_a, const __g
                 float v[16];
                 tmem_ld16(taddr + c * 16, v);
                 if (m >= M) continue;
-                tp_pre_store(v, epilogue, gate, m, n, M, N);
+                if (MAPPED) tp_pre_store(v, epilogue, gate, m, n, M, N);
                 const bool whole = vec_ok && n + 16 <= N;
                 if (epilogue == EPI_SWIGLU) {
                     if (whole) {
@@ -892,11 +894,15 @@ static TcPlan plan_tc(int M, int N, int K, int g_tc_tune_ksplit) {
     return p;
 }
 
-template <int BT>
+static bool tc_mapped(int epilogue) {
+    return epilogue == BFI_EPI_RELU_SQUARED || (epilogue == EPI_SWIGLU && g_bfi_gate.in_scale != nullptr);
+}
+
+template <int BT, bool MAPPED>
 static int launch_tc(const TcPlan& p, const CUtensorMap& mw, const CUtensorMap& ma, void* C, int c_dtype, long ldc,
                      int M, int N, int K, int epilogue, int* status, cudaStream_t stream, TcWaits waits) {
     using Cfg = TcConfig<BT>;
-    auto kernel = gemm_tcgen05_kernel<BT>;
+    auto kernel = gemm_tcgen05_kernel<BT, MAPPED>;
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Cfg::SMEM);
@@ -939,10 +945,14 @@ static int launch_tc_prefill(const void* A, long lda, const void* W, long ldw, v
     static bool configured = false;
     const int n_sm = bfi_sm_count();
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_prefill_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_prefill_kernel<1, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              (int)TP_SMEM);
         if (e == cudaSuccess)
-            e = cudaFuncSetAttribute(gemm_tcgen05_prefill_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TP_SMEM);
+            e = cudaFuncSetAttribute(gemm_tcgen05_prefill_kernel<2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TP_SMEM);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(gemm_tcgen05_prefill_kernel<1, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TP_SMEM);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(gemm_tcgen05_prefill_kernel<2, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TP_SMEM);
         if (e != cudaSuccess)
             return bfi_fail("gemm_tcgen05: cannot reserve %zu bytes of shared memory: %s", (size_t)TP_SMEM, cudaGetErrorString(e));
         configured = true;
@@ -989,12 +999,11 @@ static int launch_tc_prefill(const void* A, long lda, const void* W, long ldw, v
     // whole 16-byte stores need aligned rows: output row stride and base
     const int elem = dtype_size(c_dtype);
     const int vec_ok = ((ldc * elem) % 16 == 0 && ((uintptr_t)C & 15) == 0) ? 1 : 0;
-    if (halves == 2)
-        bfi_launch(gemm_tcgen05_prefill_kernel<2>, dim3(grid), dim3(TP_THREADS), TP_SMEM, stream, ma, mw, C, c_dtype, ldc, M, N,
-                   K, tiles_m, tiles_n, tile_n, n_stages, epilogue, g_bfi_gate, vec_ok, status, waits);
-    else
-        bfi_launch(gemm_tcgen05_prefill_kernel<1>, dim3(grid), dim3(TP_THREADS), TP_SMEM, stream, ma, mw, C, c_dtype, ldc, M, N,
-                   K, tiles_m, tiles_n, tile_n, n_stages, epilogue, g_bfi_gate, vec_ok, status, waits);
+    const bool mapped = tc_mapped(epilogue);
+    auto kernel = halves == 2 ? (mapped ? gemm_tcgen05_prefill_kernel<2, true> : gemm_tcgen05_prefill_kernel<2, false>)
+                              : (mapped ? gemm_tcgen05_prefill_kernel<1, true> : gemm_tcgen05_prefill_kernel<1, false>);
+    bfi_launch(kernel, dim3(grid), dim3(TP_THREADS), TP_SMEM, stream, ma, mw, C, c_dtype, ldc, M, N, K, tiles_m, tiles_n, tile_n,
+               n_stages, epilogue, g_bfi_gate, vec_ok, status, waits);
     return bfi_check_launch("gemm_tcgen05_prefill");
 }
 
@@ -1018,13 +1027,17 @@ static int gemm_tcgen05_launch(const void* A, long lda, const void* W, long ldw,
     if (rc) return rc;
     rc = bfi_tensor_map_bf16(A, M, K, lda, p.bt, &ma);
     if (rc) return rc;
+#define BFI_TC(BTT)                                                                                                            \
+    return tc_mapped(epilogue) ? launch_tc<BTT, true>(p, mw, ma, C, c_dtype, ldc, M, N, K, epilogue, status, stream, waits)     \
+                               : launch_tc<BTT, false>(p, mw, ma, C, c_dtype, ldc, M, N, K, epilogue, status, stream, waits)
     switch (p.bt) {
-        case 16: return launch_tc<16>(p, mw, ma, C, c_dtype, ldc, M, N, K, epilogue, status, stream, waits);
-        case 32: return launch_tc<32>(p, mw, ma, C, c_dtype, ldc, M, N, K, epilogue, status, stream, waits);
-        case 64: return launch_tc<64>(p, mw, ma, C, c_dtype, ldc, M, N, K, epilogue, status, stream, waits);
-        case 128: return launch_tc<128>(p, mw, ma, C, c_dtype, ldc, M, N, K, epilogue, status, stream, waits);
-        default: return launch_tc<256>(p, mw, ma, C, c_dtype, ldc, M, N, K, epilogue, status, stream, waits);
+        case 16: BFI_TC(16);
+        case 32: BFI_TC(32);
+        case 64: BFI_TC(64);
+        case 128: BFI_TC(128);
+        default: BFI_TC(256);
     }
+#undef BFI_TC
 }
 
 // Returns 0 on success, 1 on error, 2 when the shape is not taken (nothing launched).
