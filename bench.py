@@ -423,7 +423,7 @@ def zirivik_config(width, heads, kv, d, ff, layers):
         mixer = ret if i % 4 < 2 else (att if i % 4 == 2 else dict(att, kv_from=i - 1))
         out.append({"type": "retention" if i % 4 < 2 else "attention", "mixer": mixer, "mlp": moe if i % 2 else {"kind": "dense", "ff": ff}})
     return {"architecture": "Zirivik", "vocab": DESIGN_VOCAB, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
-            "logit_softcap": 30.0, "layers": out}
+            "logit_softcap": 50.0, "layers": out}
 
 
 def decode_breakdown(model, batch, ctx_len):

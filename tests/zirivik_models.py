@@ -162,7 +162,7 @@ def random_config(seed):
     layers, lenders = [], []
 
     def mask():
-        return rng.choice([1, 2, 9, 40, 63, 64, 65, 100, 1000]), rng.choice([0, 1, 2, 6, 63, 64, 65, 130])
+        return rng.choice([1, 2, 9, 38, 63, 64, 65, 100, 1000]), rng.choice([0, 1, 2, 7, 63, 64, 65, 130])
 
     for i in range(rng.randint(2, 6)):
         kind = rng.choice(["retention", "attention", "attention"])
@@ -191,7 +191,7 @@ def random_config(seed):
             mlp = moe(e, rng.randint(1, min(e, 4)), rng.choice([12, 20, 32, 64]), rng.choice([0.2, 1.0, 7.0]))
         layers.append((lay, mlp))
     cfg = config(rng.choice([97, 256, 333]), width, rng.choice([1e-6, 1e-5]), rng.choice([1.0, 0.5, math.sqrt(width)]),
-                 rng.choice([5.0, 30.0]), layers)
+                 rng.choice([5.0, 25.0]), layers)
     if rng.random() < 0.2:
         del cfg["logit_softcap"]
     return cfg
