@@ -63,14 +63,15 @@ struct DecodeSmem {
 
 // part_o  [seqs, n_q, max_splits, D]  float32 unnormalised outputs
 // part_ml [seqs, n_q, max_splits, 2]  float32 (running max in log2 units, running sum)
-template <int D, bool SPLIT_P>
+// CAP: the scores are soft-capped (ScoreCap)
+template <int D, bool SPLIT_P, bool CAP>
 __global__ void __launch_bounds__(AD_THREADS)
 attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out, long out_stride,
                         const int* __restrict__ block_table, int table_stride, const int* __restrict__ seq_slot,
                         const int* __restrict__ seq_start, int n_q, int n_kv, int window, int keep_first, float scale_log2, float sink_log2,
                         int head_chunks, float* __restrict__ part_o, float* __restrict__ part_ml,
-                        int* __restrict__ status, TcWaits waits) {
+                        int* __restrict__ status, TcWaits waits, const ScoreCap cap) {
     pdl_trigger();
     const uint32_t spin_limit = waits.spin_limit;
     using Smem = DecodeSmem<D>;
@@ -233,7 +234,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
                 for (int c = 0; c < 2; ++c) {
                     const int key = key0 + j * 8 + 2 * t + c;
-                    float v = s[j][r * 2 + c] * scale_log2;
+                    float v = CAP ? score_capped(s[j][r * 2 + c], cap) : s[j][r * 2 + c] * scale_log2;
                     if (!have_page || key > pos || (key < lo && key >= keep_first)) v = -INFINITY;
                     s[j][r * 2 + c] = v;
                     mx = fmaxf(mx, v);
@@ -399,7 +400,7 @@ template <int D>
 static int launch_decode(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                          const void* v_pages, long n_pages, const int* block_table, int table_stride,
                          const int* seq_slot, const int* seq_start, int n_seqs, int n_q, int n_kv, int window, int keep_first,
-                         float scale, float sink, int split_p, int max_splits, float* part_o, float* part_ml, int* status, cudaStream_t stream, TcWaits waits) {
+                         float scale, float sink, int split_p, float softcap, int max_splits, float* part_o, float* part_ml, int* status, cudaStream_t stream, TcWaits waits) {
     CUtensorMap mk, mv;
     int rc = bfi_tensor_map_bf16(k_pages, n_pages * n_kv * AD_TILE, D, D, AD_TILE, &mk);
     if (rc) return rc;
@@ -408,7 +409,8 @@ static int launch_decode(const void* q, long q_stride, void* out, long out_strid
     const int group = n_q / n_kv;
     const int head_chunks = (group + 15) / 16;
     const size_t need = DecodeSmem<D>::BYTES;
-    auto kernel = split_p ? attention_decode_kernel<D, true> : attention_decode_kernel<D, false>;
+    auto kernel = softcap > 0.0f ? (split_p ? attention_decode_kernel<D, true, true> : attention_decode_kernel<D, false, true>)
+                                 : (split_p ? attention_decode_kernel<D, true, false> : attention_decode_kernel<D, false, false>);
     if (need > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)need);
         if (e != cudaSuccess) return bfi_fail("attention_decode: cannot reserve %zu bytes of shared memory: %s", need,
@@ -419,7 +421,7 @@ static int launch_decode(const void* q, long q_stride, void* out, long out_strid
     const float sink_log2 = sink * 1.4426950408889634f;       // -inf: no sink
     bfi_launch(kernel, grid, dim3(AD_THREADS), need, stream, mk, mv, (const bf16*)q, q_stride, (bf16*)out, out_stride,
                block_table, table_stride, seq_slot, seq_start, n_q, n_kv, window, keep_first, scale_log2, sink_log2, head_chunks, part_o, part_ml,
-               status, waits);
+               status, waits, score_cap(scale, softcap));
     rc = bfi_check_launch("attention_decode");
     if (rc || max_splits == 1) return rc;
 #define BFI_MERGE(CAP)                                                                                                   \
@@ -438,10 +440,11 @@ static int launch_decode(const void* q, long q_stride, void* out, long out_strid
 // gives part_o [n_seqs*n_q*max_splits*d] and part_ml [n_seqs*n_q*max_splits*2] floats.  `status` points at
 // an int, zero before the first call, that gets BFI_STATUS_TIMEOUT when a wait for a page ran out.
 // `sink`: a score beside the keys' whose exponential joins the softmax's denominator; -infinity for none.
+// `softcap` > 0: a score becomes softcap * tanh(score / softcap) before the softmax.
 static int attention_decode_launch(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                                    const void* v_pages, long n_pages, const int* block_table, int table_stride,
                                    const int* seq_slot, const int* seq_start, int n_seqs, int n_q, int n_kv, int d,
-                                   int window, int keep_first, float scale, float sink, int split_p, int max_splits, float* part_o,
+                                   int window, int keep_first, float scale, float sink, int split_p, float softcap, int max_splits, float* part_o,
                                    float* part_ml, int* status, cudaStream_t stream, TcWaits waits) {
     BFI_REQUIRE(n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_decode: %d query heads do not divide into %d kv heads",
                 n_q, n_kv);
@@ -455,10 +458,10 @@ static int attention_decode_launch(const void* q, long q_stride, void* out, long
     if (max_splits > 1) BFI_REQUIRE(part_o && part_ml, "attention_decode: split runs need the scratch buffers");
     if (d == 64)
         return launch_decode<64>(q, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
-                                 seq_slot, seq_start, n_seqs, n_q, n_kv, window, keep_first, scale, sink, split_p, max_splits, part_o, part_ml,
+                                 seq_slot, seq_start, n_seqs, n_q, n_kv, window, keep_first, scale, sink, split_p, softcap, max_splits, part_o, part_ml,
                                  status, stream, waits);
     return launch_decode<128>(q, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride, seq_slot,
-                              seq_start, n_seqs, n_q, n_kv, window, keep_first, scale, sink, split_p, max_splits, part_o, part_ml, status,
+                              seq_start, n_seqs, n_q, n_kv, window, keep_first, scale, sink, split_p, softcap, max_splits, part_o, part_ml, status,
                               stream, waits);
 }
 
@@ -466,9 +469,9 @@ extern "C" int bfi_attention_decode_bf16(const void* q, long q_stride, void* out
                                          const void* v_pages, long n_pages, const int* block_table, int table_stride,
                                          const int* seq_slot, const int* seq_start, int n_seqs, int n_q, int n_kv,
                                          int d, int window, int keep_first, float scale, float sink, int split_p,
-                                         int max_splits, float* part_o, float* part_ml, int* status, cudaStream_t stream) {
+                                         float softcap, int max_splits, float* part_o, float* part_ml, int* status, cudaStream_t stream) {
     return attention_decode_launch(q, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
-                                   seq_slot, seq_start, n_seqs, n_q, n_kv, d, window, keep_first, scale, sink, split_p, max_splits, part_o,
+                                   seq_slot, seq_start, n_seqs, n_q, n_kv, d, window, keep_first, scale, sink, split_p, softcap, max_splits, part_o,
                                    part_ml, status, stream, tc_waits_default());
 }
 
@@ -485,7 +488,7 @@ extern "C" int bfi_attention_decode_bf16_wait_probe(const void* q, long q_stride
                                                     cudaStream_t stream) {
     BFI_REQUIRE(spin_limit > 0 && spin_limit <= TC_SPIN_LIMIT, "attention_decode probe: spin limit out of range");
     return attention_decode_launch(q, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
-                                   seq_slot, seq_start, n_seqs, n_q, n_kv, d, window, 0, scale, -INFINITY, 0, max_splits, part_o, part_ml,
+                                   seq_slot, seq_start, n_seqs, n_q, n_kv, d, window, 0, scale, -INFINITY, 0, 0.0f, max_splits, part_o, part_ml,
                                    status, stream, TcWaits{spin_limit, hold_producer ? 1 : 0});
 }
 

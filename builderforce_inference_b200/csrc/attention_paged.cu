@@ -12,6 +12,7 @@
 // `has_sink`: the softmax's denominator carries one more term, exp(sink), a score that every
 // query sees and that has no value: p_j = exp(s_j) / (exp(sink) + sum_i exp(s_i)); the sink is one
 // number (`has_sink` 1) or one float32 per query head (`has_sink` 2, `sinks`).
+// `softcap` > 0: a score becomes softcap * tanh(score / softcap) before the softmax (a sink does not).
 // Keys have `d` values per head, values `dv` (the cache's value pages are laid out by `dv`).
 // Without value pages (`v_pages` null) a key's first `dv` values are its value: the cache of a
 // latent attention holds one row per token that serves as both.
@@ -35,7 +36,7 @@ attention_paged_kernel(const T* __restrict__ q, long q_stride, T* __restrict__ o
                        const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_seqlens,
                        const int* __restrict__ seq_slot, const int* __restrict__ seq_start, int n_q, int n_kv, int d,
                        int dv, int gh, int head_chunks, int window, int keep_first, int chunk, float scale, int has_sink,
-                       float sink, const float* __restrict__ sinks) {
+                       float sink, const float* __restrict__ sinks, float softcap) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ float smem[];
@@ -139,6 +140,7 @@ attention_paged_kernel(const T* __restrict__ q, long q_stride, T* __restrict__ o
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const bool valid = row_ok[i] && page >= 0 && key <= row_pos[i] && (key >= row_lo[i] || key < keep_first);
+            if (softcap > 0.0f) s[i] = softcap * tanhf(s[i] / softcap);
             const float sc = valid ? s[i] : -INFINITY;
             const float m_tile = warp_max(sc);
             if (m_tile == -INFINITY) continue;   // no key of this tile is visible to the row (uniform in the warp)
@@ -186,7 +188,7 @@ static int launch_attention(const void* q, long q_stride, void* out, long out_st
                             const void* v_pages, const int* block_table, int table_stride, const int* cu_seqlens,
                             const int* seq_slot, const int* seq_start, int n_seqs, int max_tokens, int n_q, int n_kv,
                             int d, int dv, int window, int keep_first, int chunk, float scale, int has_sink, float sink,
-                            const float* sinks, cudaStream_t stream) {
+                            const float* sinks, float softcap, cudaStream_t stream) {
     const int group = n_q / n_kv;
     int gh = 1;
     while (gh < group && gh < 8) gh *= 2;
@@ -204,7 +206,7 @@ static int launch_attention(const void* q, long q_stride, void* out, long out_st
     }
     bfi_launch(kernel, dim3(grid), dim3(ATT_WARPS * 32), smem, stream, (const T*)q, q_stride, (T*)out, out_stride, (const T*)k_pages,
                                                    (const T*)v_pages, block_table, table_stride, cu_seqlens, seq_slot,
-                                                   seq_start, n_q, n_kv, d, dv, gh, head_chunks, window, keep_first, chunk, scale, has_sink, sink, sinks);
+                                                   seq_start, n_q, n_kv, d, dv, gh, head_chunks, window, keep_first, chunk, scale, has_sink, sink, sinks, softcap);
     return bfi_check_launch("attention_paged");
 }
 
@@ -213,12 +215,12 @@ static int dispatch_nc(int nc, const void* q, long q_stride, void* out, long out
                        const void* v_pages, const int* block_table, int table_stride, const int* cu_seqlens,
                        const int* seq_slot, const int* seq_start, int n_seqs, int max_tokens, int n_q, int n_kv, int d,
                        int dv, int window, int keep_first, int chunk, float scale, int has_sink, float sink,
-                       const float* sinks, cudaStream_t stream) {
+                       const float* sinks, float softcap, cudaStream_t stream) {
 #define BFI_ATT_CASE(N)                                                                                              \
     case N:                                                                                                          \
         return launch_attention<T, N>(q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride,     \
                                       cu_seqlens, seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, \
-                                      keep_first, chunk, scale, has_sink, sink, sinks, stream);
+                                      keep_first, chunk, scale, has_sink, sink, sinks, softcap, stream);
     switch (nc) {
         BFI_ATT_CASE(1)
         BFI_ATT_CASE(2)
@@ -238,7 +240,7 @@ extern "C" int bfi_attention_paged(const void* q, int dtype, long q_stride, void
                                    const void* k_pages, const void* v_pages, const int* block_table, int table_stride,
                                    const int* cu_seqlens, const int* seq_slot, const int* seq_start, int n_seqs,
                                    int max_tokens, int n_q, int n_kv, int d, int dv, int window, int keep_first, int chunk, float scale,
-                                   int has_sink, float sink, const float* sinks, cudaStream_t stream) {
+                                   int has_sink, float sink, const float* sinks, float softcap, cudaStream_t stream) {
     BFI_REQUIRE(dtype_ok(dtype), "attention_paged: unknown dtype code %d", dtype);
     BFI_REQUIRE(n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_paged: %d query heads do not divide into %d kv heads",
                 n_q, n_kv);
@@ -258,7 +260,7 @@ extern "C" int bfi_attention_paged(const void* q, int dtype, long q_stride, void
     if (nc > 8) nc = 16;
     if (dtype == BFI_F32)
         return dispatch_nc<float>(nc, q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride,
-                                  cu_seqlens, seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, keep_first, chunk, scale, has_sink, sink, sinks, stream);
+                                  cu_seqlens, seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, keep_first, chunk, scale, has_sink, sink, sinks, softcap, stream);
     return dispatch_nc<bf16>(nc, q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride, cu_seqlens,
-                             seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, keep_first, chunk, scale, has_sink, sink, sinks, stream);
+                             seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, d, dv, window, keep_first, chunk, scale, has_sink, sink, sinks, softcap, stream);
 }

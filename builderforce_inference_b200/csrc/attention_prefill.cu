@@ -14,14 +14,15 @@
 
 #define AP_QROWS 64
 
-template <int D>
+// CAP: the scores are soft-capped (ScoreCap)
+template <int D, bool CAP>
 __global__ void __launch_bounds__(AD_THREADS)
 attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __restrict__ out, long out_stride,
                          const bf16* __restrict__ k_pages, const bf16* __restrict__ v_pages,
                          const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_seqlens,
                          const int* __restrict__ seq_slot, const int* __restrict__ seq_start, int n_q, int n_kv,
                          int window, int keep_first, int chunk, float scale_log2, float sink_log2, const float* __restrict__ sinks,
-                         int split_p) {
+                         int split_p, const ScoreCap cap) {
     pdl_trigger();
     pdl_wait();
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -159,7 +160,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __rest
                 for (int j = 0; j < 8; ++j)
 #pragma unroll
                     for (int c = 0; c < 2; ++c) {
-                        float v = s[j][r * 2 + c] * scale_log2;
+                        float v = CAP ? score_capped(s[j][r * 2 + c], cap) : s[j][r * 2 + c] * scale_log2;
                         if (need_mask) {
                             const int key = key_lo + j * 8 + 2 * t + c;
                             if (key > pos_r[r] || (key < lo_r[r] && key >= keep_first)) v = -INFINITY;
@@ -242,14 +243,14 @@ attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __rest
     }
 }
 
-template <int D>
+template <int D, bool CAP>
 static int launch_prefill(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                           const void* v_pages, const int* block_table, int table_stride, const int* cu_seqlens,
                           const int* seq_slot, const int* seq_start, int n_seqs, int max_tokens, int n_q, int n_kv,
                           int window, int keep_first, int chunk, float scale, float sink, const float* sinks, int split_p,
-                          cudaStream_t stream) {
+                          float softcap, cudaStream_t stream) {
     const size_t smem = (size_t)(AP_QROWS * D + 4 * AD_TILE * D) * sizeof(bf16);
-    auto kernel = attention_prefill_kernel<D>;
+    auto kernel = attention_prefill_kernel<D, CAP>;
     if (smem > 48 * 1024) {
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return bfi_fail("attention_prefill: cannot reserve %zu bytes of shared memory: %s", smem,
@@ -258,7 +259,8 @@ static int launch_prefill(const void* q, long q_stride, void* out, long out_stri
     dim3 grid((max_tokens + AP_QROWS - 1) / AP_QROWS, n_q, n_seqs);
     bfi_launch(kernel, grid, dim3(AD_THREADS), smem, stream, (const bf16*)q, q_stride, (bf16*)out, out_stride,
                (const bf16*)k_pages, (const bf16*)v_pages, block_table, table_stride, cu_seqlens, seq_slot, seq_start, n_q,
-               n_kv, window, keep_first, chunk, scale * 1.4426950408889634f, sink * 1.4426950408889634f, sinks, split_p);
+               n_kv, window, keep_first, chunk, scale * 1.4426950408889634f, sink * 1.4426950408889634f, sinks, split_p,
+               score_cap(scale, softcap));
     return bfi_check_launch("attention_prefill");
 }
 
@@ -267,12 +269,13 @@ static int launch_prefill(const void* q, long q_stride, void* out, long out_stri
 // `sinks` (float32, one per query head) takes its place when given.  `chunk` > 0: a token reads only
 // the keys of its own block of `chunk` consecutive positions, blocks counted from position 0.
 // `split_p`: the softmax's weights enter the second product as two bfloat16 terms (the rounded weight
-// and what the rounding left over), for designs whose attention weights are float32 by rule.
+// and what the rounding left over), for designs whose attention weights are float32 by rule.  `softcap` > 0:
+// a score becomes softcap * tanh(score / softcap) before the mask and the softmax.
 extern "C" int bfi_attention_prefill_bf16(const void* q, long q_stride, void* out, long out_stride, const void* k_pages,
                                           const void* v_pages, const int* block_table, int table_stride,
                                           const int* cu_seqlens, const int* seq_slot, const int* seq_start, int n_seqs,
                                           int max_tokens, int n_q, int n_kv, int d, int window, int keep_first, int chunk, float scale,
-                                          float sink, const float* sinks, int split_p, cudaStream_t stream) {
+                                          float sink, const float* sinks, int split_p, float softcap, cudaStream_t stream) {
     BFI_REQUIRE(n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_prefill: %d query heads do not divide into %d kv heads",
                 n_q, n_kv);
     BFI_REQUIRE(window >= 0 && chunk >= 0, "attention_prefill: negative window or chunk");
@@ -282,11 +285,15 @@ extern "C" int bfi_attention_prefill_bf16(const void* q, long q_stride, void* ou
     if (q_stride % 8 != 0 || out_stride % 2 != 0 || ((uintptr_t)q & 15) || ((uintptr_t)out & 3) || n_seqs > 65535 ||
         n_q > 65535)
         return 2;
-    if (d == 64)
-        return launch_prefill<64>(q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride, cu_seqlens,
-                                  seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, window, keep_first, chunk, scale, sink, sinks, split_p,
-                                  stream);
-    return launch_prefill<128>(q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride, cu_seqlens,
-                               seq_slot, seq_start, n_seqs, max_tokens, n_q, n_kv, window, keep_first, chunk, scale, sink, sinks, split_p,
-                               stream);
+#define BFI_PREFILL(DD, CC)                                                                                                      \
+    return launch_prefill<DD, CC>(q, q_stride, out, out_stride, k_pages, v_pages, block_table, table_stride, cu_seqlens, seq_slot, \
+                                  seq_start, n_seqs, max_tokens, n_q, n_kv, window, keep_first, chunk, scale, sink, sinks, split_p, \
+                                  softcap, stream)
+    if (softcap > 0.0f) {
+        if (d == 64) BFI_PREFILL(64, true);
+        BFI_PREFILL(128, true);
+    }
+    if (d == 64) BFI_PREFILL(64, false);
+    BFI_PREFILL(128, false);
+#undef BFI_PREFILL
 }

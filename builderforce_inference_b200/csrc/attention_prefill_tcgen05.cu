@@ -175,14 +175,15 @@ struct FtItem {
 };
 
 // KEEP: there may be kept first positions (without them the kernel is the one for plain windows).
-template <int D, bool SPLIT_P, bool KEEP>
+// CAP: the scores are soft-capped as they are read; they are then in the exponent's units (scale_log2 is 1).
+template <int D, bool SPLIT_P, bool KEEP, bool CAP>
 __global__ void __launch_bounds__(FT_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                             const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, long out_stride,
                             const int* __restrict__ block_table, int table_stride, const int* __restrict__ cu_seqlens,
                             const int* __restrict__ seq_slot, const int* __restrict__ seq_start, int n_seqs, int max_tiles,
                             int n_q, int n_kv, int window, int keep_first, float scale_log2, float sink_log2, uint32_t v_lbo, uint32_t v_sbo,
-                            int* __restrict__ status, int* __restrict__ counters, TcWaits waits) {
+                            int* __restrict__ status, int* __restrict__ counters, TcWaits waits, const ScoreCap cap) {
     const uint32_t spin_limit = waits.spin_limit;
     constexpr int BOXES = D / 64;
     constexpr int TILE_BYTES = BOXES * FT_BOX_BYTES;       // a Q tile, a K tile or a V tile
@@ -540,6 +541,10 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                 for (int c = 0; c < FT_KEYS / 32; ++c) tmem_ld32(s_addr + c * 32, s + c * 32);
                 tmem_wait_ld();
+                if (CAP) {
+#pragma unroll
+                    for (int e = 0; e < FT_KEYS; ++e) s[e] = score_capped(s[e], cap);
+                }
                 const int key0 = j * FT_KEYS;
                 const bool masked = key0 + FT_KEYS - 1 > p0 || key0 + FT_KEYS - 1 > seq_hi ||
                                     (window > 0 && key0 < p0 + FT_ROWS - 1 - window + 1);
@@ -664,11 +669,11 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     BFI_TRACE_END();
 }
 
-template <int D, bool SPLIT_P, bool KEEP>
+template <int D, bool SPLIT_P, bool KEEP, bool CAP>
 static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out_stride, const void* k_pages,
                              const void* v_pages, long n_pages, const int* block_table, int table_stride,
                              const int* cu_seqlens, const int* seq_slot, const int* seq_start, int n_seqs, long n_tokens,
-                             int max_seq_tokens, int n_q, int n_kv, int window, int keep_first, float scale, float sink, int* status,
+                             int max_seq_tokens, int n_q, int n_kv, int window, int keep_first, float scale, float sink, float softcap, int* status,
                              cudaStream_t stream, TcWaits waits) {
     CUtensorMap mq, mk, mv;
     int rc = bfi_tensor_map_bf16(qkv, n_tokens, (long)n_q * D, q_stride, FT_ROWS, &mq);
@@ -681,7 +686,7 @@ static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out
     // at least half an SM's shared memory, so that two blocks never share one SM's tensor memory
     const size_t tiles = (size_t)6 * TILE_BYTES + 1024 + 512 + FT_META_SEQS * sizeof(int4) + 4 * 4096;
     const size_t smem = tiles > 120 * 1024 ? tiles : 120 * 1024;
-    auto kernel = attention_prefill_tc_kernel<D, SPLIT_P, KEEP>;
+    auto kernel = attention_prefill_tc_kernel<D, SPLIT_P, KEEP, CAP>;
     static bool configured = false;
     const int n_sm = bfi_sm_count();
     if (!configured) {
@@ -696,8 +701,9 @@ static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out
     const long items = (long)max_tiles * n_seqs * n_q;
     dim3 grid((unsigned)(items < n_sm ? items : n_sm));      // one block per SM, each drawing items until none is left
     bfi_launch(kernel, grid, dim3(FT_THREADS), smem, stream, mq, mk, mv, (bf16*)out, out_stride, block_table, table_stride,
-               cu_seqlens, seq_slot, seq_start, n_seqs, max_tiles, n_q, n_kv, window, keep_first, scale * 1.4426950408889634f,
-               sink * 1.4426950408889634f, (uint32_t)lbo, (uint32_t)sbo, status, status + 1, waits);
+               cu_seqlens, seq_slot, seq_start, n_seqs, max_tiles, n_q, n_kv, window, keep_first,
+               CAP ? 1.0f : scale * 1.4426950408889634f, sink * 1.4426950408889634f, (uint32_t)lbo, (uint32_t)sbo, status, status + 1, waits,
+               score_cap(scale, softcap));
     return bfi_check_launch("attention_prefill_tcgen05");
 }
 
@@ -708,12 +714,13 @@ static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out
 // zero before the first call: [0] gets BFI_STATUS_TIMEOUT when a wait ran out, [1] and [2] are
 // the counters of tickets drawn and blocks finished, which every launch leaves at zero again; two
 // launches that may run at the same time need status words of their own.  `sink`: a score beside the
-// keys' whose exponential joins the softmax's denominator; -infinity for none.
+// keys' whose exponential joins the softmax's denominator; -infinity for none.  `softcap` > 0: a score becomes
+// softcap * tanh(score / softcap) before the mask and the softmax.
 static int attention_prefill_tc_launch(const void* qkv, long q_stride, void* out, long out_stride, const void* k_pages,
                                        const void* v_pages, long n_pages, const int* block_table, int table_stride,
                                        const int* cu_seqlens, const int* seq_slot, const int* seq_start, int n_seqs,
                                        long n_tokens, int max_seq_tokens, int n_q, int n_kv, int d, int window, int keep_first,
-                                       float scale, float sink, int split_p, int* status, cudaStream_t stream, TcWaits waits) {
+                                       float scale, float sink, int split_p, float softcap, int* status, cudaStream_t stream, TcWaits waits) {
     BFI_REQUIRE(n_q > 0 && n_kv > 0 && n_q % n_kv == 0, "attention_prefill_tcgen05: %d query heads do not divide into %d kv heads",
                 n_q, n_kv);
     BFI_REQUIRE(window >= 0 && status != nullptr, "attention_prefill_tcgen05: bad window or no status word");
@@ -724,10 +731,17 @@ static int attention_prefill_tc_launch(const void* qkv, long q_stride, void* out
         ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15) || (long)((max_seq_tokens + FT_ROWS - 1) / FT_ROWS) * n_seqs * n_q > 0x3fffffffL)
         return 2;
     if (n_pages * n_kv * FT_PAGE > 0x7fffffffL) return 2;       // TMA coordinates are 32-bit
-#define BFI_PREFILL_TC(DD, SP, KP)                                                                                              \
-    return launch_prefill_tc<DD, SP, KP>(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,   \
+#define BFI_PREFILL_TC_CAP(DD, SP, KP, CC)                                                                                      \
+    return launch_prefill_tc<DD, SP, KP, CC>(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,   \
                                      cu_seqlens, seq_slot, seq_start, n_seqs, n_tokens, max_seq_tokens, n_q, n_kv, window,   \
-                                     keep_first, scale, sink, status, stream, waits)
+                                     keep_first, scale, sink, softcap, status, stream, waits)
+#define BFI_PREFILL_TC(DD, SP, KP) BFI_PREFILL_TC_CAP(DD, SP, KP, false)
+    if (softcap > 0.0f) {
+        if (split_p && d == 64) BFI_PREFILL_TC_CAP(64, true, true, true);
+        if (split_p) BFI_PREFILL_TC_CAP(128, true, true, true);
+        if (d == 64) BFI_PREFILL_TC_CAP(64, false, true, true);
+        BFI_PREFILL_TC_CAP(128, false, true, true);
+    }
     if (split_p) {
         if (d == 64) BFI_PREFILL_TC(64, true, true);
         BFI_PREFILL_TC(128, true, true);
@@ -739,6 +753,7 @@ static int attention_prefill_tc_launch(const void* qkv, long q_stride, void* out
     if (d == 64) BFI_PREFILL_TC(64, false, false);
     BFI_PREFILL_TC(128, false, false);
 #undef BFI_PREFILL_TC
+#undef BFI_PREFILL_TC_CAP
 }
 
 extern "C" int bfi_attention_prefill_tcgen05_bf16(const void* qkv, long q_stride, void* out, long out_stride,
@@ -746,10 +761,10 @@ extern "C" int bfi_attention_prefill_tcgen05_bf16(const void* qkv, long q_stride
                                                   const int* block_table, int table_stride, const int* cu_seqlens,
                                                   const int* seq_slot, const int* seq_start, int n_seqs, long n_tokens,
                                                   int max_seq_tokens, int n_q, int n_kv, int d, int window, int keep_first,
-                                                  float scale, float sink, int split_p, int* status, cudaStream_t stream) {
+                                                  float scale, float sink, int split_p, float softcap, int* status, cudaStream_t stream) {
     return attention_prefill_tc_launch(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
                                        cu_seqlens, seq_slot, seq_start, n_seqs, n_tokens, max_seq_tokens, n_q, n_kv, d, window,
-                                       keep_first, scale, sink, split_p, status, stream, tc_waits_default());
+                                       keep_first, scale, sink, split_p, softcap, status, stream, tc_waits_default());
 }
 
 // For the tests of the time-out path: the same launch, but every bounded wait gives up after
@@ -769,7 +784,7 @@ extern "C" int bfi_attention_prefill_tcgen05_bf16_wait_probe(const void* qkv, lo
                 spin_limit);
     return attention_prefill_tc_launch(qkv, q_stride, out, out_stride, k_pages, v_pages, n_pages, block_table, table_stride,
                                        cu_seqlens, seq_slot, seq_start, n_seqs, n_tokens, max_seq_tokens, n_q, n_kv, d, window,
-                                       0, scale, -INFINITY, 0, status, stream, TcWaits{spin_limit, hold_producer ? 1 : 0});
+                                       0, scale, -INFINITY, 0, 0.0f, status, stream, TcWaits{spin_limit, hold_producer ? 1 : 0});
 }
 
 BFI_TRACE_EXPORT(attention_prefill_tcgen05)

@@ -248,5 +248,21 @@ __device__ __forceinline__ float gate_mul_fast(float g, float u, const GateAct a
     return __fdividef(g, 1.0f + __expf(-a.alpha * g)) * (u + a.shift);
 }
 
+// Soft-capped attention scores, cap * tanh(s / cap), as the bfloat16 attention kernels apply them to their
+// float32 scores: `in` takes a product of query and key to s / cap, `out` is the cap in the softmax's units
+// (times log2 e).  tanh(x) = 1 - 2 / (1 + e^2x): absolute error of a few float32 roundings of 1, so a score is
+// right to about 1e-6 of the cap; e^2x overflowing to infinity gives 1, vanishing gives -1.
+struct ScoreCap {
+    float in, out;
+};
+static inline ScoreCap score_cap(float scale, float cap) {
+    ScoreCap c = {0.0f, 0.0f};
+    if (cap > 0.0f) c.in = scale / cap, c.out = cap * 1.4426950408889634f;
+    return c;
+}
+__device__ __forceinline__ float score_capped(float qk, const ScoreCap c) {
+    return c.out * (1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * (c.in * qk))));
+}
+
 static inline int dtype_size(int dtype) { return dtype == BFI_F32 ? 4 : 2; }
 static inline bool dtype_ok(int dtype) { return dtype == BFI_F32 || dtype == BFI_BF16; }

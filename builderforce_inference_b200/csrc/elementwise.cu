@@ -11,36 +11,36 @@
 #include "common.cuh"
 
 // ------------------------------------------------------------------------------------------
-// embedding: out[t, :] = table[ids[t], :] * scale   (out is the float32 residual stream)
+// embedding: out[t, c, :] = table[ids[t], :] * scale for every copy c   (out is the float32 residual stream)
 // ------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void embed_rows_kernel(const T* __restrict__ table, const int* __restrict__ ids,
-                                  float* __restrict__ out, int width, int vocab, float scale, int* status) {
+                                  float* __restrict__ out, int width, int vocab, float scale, int copies, int* status) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
     const int id = ids[t];
-    float* o = out + (size_t)t * width;
-    if (id < 0 || id >= vocab) {
-        if (threadIdx.x == 0 && status) atomicOr(status, BFI_STATUS_BAD_TOKEN);
-        for (int j = threadIdx.x; j < width; j += blockDim.x) o[j] = 0.0f;
-        return;
+    const bool known = id >= 0 && id < vocab;
+    float* o = out + (size_t)t * width * copies;
+    if (!known && threadIdx.x == 0 && status) atomicOr(status, BFI_STATUS_BAD_TOKEN);
+    const T* row = table + (size_t)(known ? id : 0) * width;
+    for (int j = threadIdx.x; j < width; j += blockDim.x) {
+        const float v = known ? to_f32(row[j]) * scale : 0.0f;
+        for (int c = 0; c < copies; ++c) o[(size_t)c * width + j] = v;
     }
-    const T* row = table + (size_t)id * width;
-    for (int j = threadIdx.x; j < width; j += blockDim.x) o[j] = to_f32(row[j]) * scale;
 }
 
-extern "C" int bfi_embed_rows(const void* table, int table_dtype, const int* ids, float* out,
-                              int n_tokens, int width, int vocab, float scale, int* status, cudaStream_t stream) {
+extern "C" int bfi_embed_rows(const void* table, int table_dtype, const int* ids, float* out, int n_tokens, int width, int vocab,
+                              float scale, int copies, int* status, cudaStream_t stream) {
     BFI_REQUIRE(dtype_ok(table_dtype), "embed_rows: unknown table dtype code %d", table_dtype);
-    BFI_REQUIRE(n_tokens >= 0 && width > 0 && vocab > 0, "embed_rows: bad sizes tokens=%d width=%d vocab=%d",
-                n_tokens, width, vocab);
+    BFI_REQUIRE(n_tokens >= 0 && width > 0 && vocab > 0 && copies > 0, "embed_rows: bad sizes tokens=%d width=%d vocab=%d copies=%d",
+                n_tokens, width, vocab, copies);
     if (n_tokens == 0) return 0;
     const int threads = width >= 1024 ? 256 : 128;
     if (table_dtype == BFI_F32)
-        bfi_launch(embed_rows_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, (const float*)table, ids, out, width, vocab, scale, status);
+        bfi_launch(embed_rows_kernel<float>, dim3(n_tokens), dim3(threads), 0, stream, (const float*)table, ids, out, width, vocab, scale, copies, status);
     else
-        bfi_launch(embed_rows_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, stream, (const bf16*)table, ids, out, width, vocab, scale, status);
+        bfi_launch(embed_rows_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, stream, (const bf16*)table, ids, out, width, vocab, scale, copies, status);
     return bfi_check_launch("embed_rows");
 }
 

@@ -59,6 +59,8 @@ def expected_tensors(spec: ModelSpec) -> Dict[str, ParamSpec]:
 class Decoder:
     def __init__(self, spec: ModelSpec, runtime: Runtime):
         _validate_schedule(spec)
+        if spec.streams < 1 or (spec.streams > 1 and spec.input_parts):
+            raise ValueError("input parts add to a single residual stream")
         self.spec = spec
         self.runtime = runtime
         self.blocks: List[Block] = [BLOCKS.build(layer.block) for layer in spec.layers]
@@ -145,10 +147,15 @@ class Decoder:
         return out
 
     # ---- compute ---------------------------------------------------------------------
+    def residual(self, ctx) -> torch.Tensor:
+        """The step's residual stream, float32 ``[tokens, streams * width]``: a token's copies side by side."""
+        return ctx.rows("residual", self.spec.streams * self.spec.width, torch.float32)
+
     def embed(self, ctx, cache=None) -> torch.Tensor:
         """The embedded tokens, with what the input parts add; ``cache`` holds their per-sequence state."""
-        x = ctx.rows("residual", self.spec.width, torch.float32)
-        ops.embed_rows(self.embedding, ctx.token_ids[:ctx.n_tokens], x, ctx.status, float(self.spec.embedding_scale))
+        x = self.residual(ctx)
+        ops.embed_rows(self.embedding, ctx.token_ids[:ctx.n_tokens], x, ctx.status, float(self.spec.embedding_scale),
+                       self.spec.streams)
         for j, part in enumerate(self.input_parts):
             if cache is None:
                 raise RuntimeError("this model's input parts keep per-sequence state: embed() needs the cache")
@@ -166,10 +173,15 @@ class Decoder:
             self.blocks[self.spec.schedule[i].layer].forward(ctx, x, cache.run_cache(i))
         ctx.extras.pop("outnorm.input", None)
         ctx.extras.pop("sandwich.input", None)
+        ctx.extras.pop("hyper.input", None)
 
     def logits(self, ctx, x: torch.Tensor, rows: torch.Tensor, out: torch.Tensor) -> None:
-        """Final norm and head at the given rows of ``x``; ``out`` is float32 ``[len(rows), vocab]``."""
-        h = self.final_norm.forward(ctx, x, rows, tag="head.norm")
+        """Final norm and head at the given rows of ``x``; ``out`` is float32 ``[len(rows), vocab]``.  Where the
+        residual stream is held several times, the copies' sum is normed."""
+        if self.spec.streams > 1:
+            h = self.final_norm.forward_streams(ctx, x, self.spec.streams, None, rows, tag="head.norm")
+        else:
+            h = self.final_norm.forward(ctx, x, rows, tag="head.norm")
         linear(h, self.head, out, EPI_STORE)
         if self.spec.logit_scale != 1.0:
             ops.scale_rows(out, float(self.spec.logit_scale))

@@ -208,7 +208,7 @@ class _DecodeGraphs:
         return ctx
 
     def run_ops(self, engine: "Engine", ctx: StepContext, ops) -> None:
-        x = ctx.rows("residual", engine.spec.width, torch.float32)
+        x = engine.decoder.residual(ctx)
         for op in ops:
             if op[0] == "embed":
                 engine.decoder.embed(ctx, engine.cache)

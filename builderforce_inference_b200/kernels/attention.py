@@ -5,9 +5,10 @@ from __future__ import annotations
 import torch
 
 
-def attend(ctx, qkv, out, kv, n_heads: int, scale: float, sink=None, exact_weights: bool = False) -> bool:
+def attend(ctx, qkv, out, kv, n_heads: int, scale: float, sink=None, exact_weights: bool = False,
+           softcap=None) -> bool:
     """``exact_weights``: the design wants its attention weights in float32; only kernels that keep
-    them so (in effect) are chosen."""
+    them so (in effect) are chosen.  ``softcap``: the cap on the scores, or None."""
     if qkv.dtype != torch.bfloat16:
         return False
     if not kv.plain or isinstance(sink, torch.Tensor):
@@ -19,11 +20,12 @@ def attend(ctx, qkv, out, kv, n_heads: int, scale: float, sink=None, exact_weigh
         if isinstance(sink, torch.Tensor) and (sink.dtype != torch.float32 or not sink.is_contiguous()):
             return False
         from . import fast_ops
-        return fast_ops.attention_prefill_bf16(ctx, qkv, out, kv, n_heads, scale, sink, exact_weights)
+        return fast_ops.attention_prefill_bf16(ctx, qkv, out, kv, n_heads, scale, sink, exact_weights, softcap)
     from . import fast_ops
     if ctx.max_seq_tokens == 1 and ctx.n_tokens == ctx.n_seqs:
-        return fast_ops.attention_decode_bf16(ctx, qkv, out, kv, n_heads, scale, sink=sink, exact_weights=exact_weights)
+        return fast_ops.attention_decode_bf16(ctx, qkv, out, kv, n_heads, scale, sink=sink, exact_weights=exact_weights,
+                                              softcap=softcap)
     if ctx.max_seq_tokens >= fast_ops.TCGEN05_ATTENTION_MIN_TOKENS and \
-            fast_ops.attention_prefill_tcgen05_bf16(ctx, qkv, out, kv, n_heads, scale, sink, exact_weights):
+            fast_ops.attention_prefill_tcgen05_bf16(ctx, qkv, out, kv, n_heads, scale, sink, exact_weights, softcap):
         return True
-    return fast_ops.attention_prefill_bf16(ctx, qkv, out, kv, n_heads, scale, sink, exact_weights)
+    return fast_ops.attention_prefill_bf16(ctx, qkv, out, kv, n_heads, scale, sink, exact_weights, softcap)

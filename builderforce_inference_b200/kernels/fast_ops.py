@@ -8,7 +8,8 @@ from ctypes import c_float, c_int, c_long
 import torch
 
 from .library import KernelError, library
-from .ops import LIGHT_ACT_SILU, _ptr, _rows_2d, _stream, dtype_code, rotation_args
+from .ops import (LIGHT_ACT_SILU, _ptr, _rows_2d, _stream, check_memory, check_memory_gates, dtype_code,
+                  rotation_args)
 
 SKINNY_MAX_ROWS = 64
 
@@ -188,9 +189,9 @@ def _sink(sink) -> c_float:
 
 
 def attention_decode_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads: int, scale: float,
-                          probe=None, sink=None, exact_weights: bool = False) -> bool:
+                          probe=None, sink=None, exact_weights: bool = False, softcap=None) -> bool:
     """One new token per sequence over its cached pages, which arrive by TMA: the cache must be
-    contiguous.  ``exact_weights``: as ``attention_prefill_bf16``.  A wait for a page that ran out shows in ``tc_status``.  ``probe``: (polls, hold
+    contiguous.  ``exact_weights``, ``softcap``: as ``attention_prefill_bf16``.  A wait for a page that ran out shows in ``tc_status``.  ``probe``: (polls, hold
     the producer), for ``attention_decode_wait_probe``."""
     d = kv.head_dim
     if d not in (64, 128) or qkv.dtype != torch.bfloat16 or kv.k.dtype != torch.bfloat16:
@@ -215,7 +216,7 @@ def attention_decode_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads
     tail = [c_int(max_splits), _ptr(part_o), _ptr(part_ml), _ptr(tc_status(qkv.device))]
     if probe is None:
         return library("fast").call_optional("bfi_attention_decode_bf16", *args, c_int(kv.keep_first), c_float(scale),
-                                             _sink(sink), c_int(1 if exact_weights else 0), *tail, _stream())
+                                             _sink(sink), c_int(1 if exact_weights else 0), c_float(softcap or 0.0), *tail, _stream())
     args += [c_float(scale)] + tail
     return library("fast").call_optional("bfi_attention_decode_bf16_wait_probe", *args, c_int(int(probe[0])),
                                          c_int(1 if probe[1] else 0), _stream())
@@ -229,9 +230,10 @@ def attention_decode_wait_probe(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n
 
 
 def attention_prefill_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads: int, scale: float, sink=None,
-                           exact_weights: bool = False) -> bool:
+                           exact_weights: bool = False, softcap=None) -> bool:
     """Tensor-core attention for steps that bring more than one token per sequence.
-    ``exact_weights``: the softmax's weights enter the second product as two bfloat16 terms."""
+    ``exact_weights``: the softmax's weights enter the second product as two bfloat16 terms.
+    ``softcap``: a score becomes ``softcap * tanh(score / softcap)`` before the softmax (None: as it is)."""
     d = kv.head_dim
     if d not in (64, 128) or kv.value_dim != d or qkv.dtype != torch.bfloat16 or kv.k.dtype != torch.bfloat16:
         return False
@@ -241,7 +243,7 @@ def attention_prefill_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_head
         _ptr(kv.v), _ptr(kv.block_table), c_int(kv.block_table.stride(0)), _ptr(ctx.cu_seqlens), _ptr(ctx.seq_slot),
         _ptr(ctx.seq_start), c_int(ctx.n_seqs), c_int(ctx.max_seq_tokens), c_int(n_heads), c_int(kv.n_kv_heads),
         c_int(d), c_int(kv.window or 0), c_int(kv.keep_first), c_int(kv.chunk or 0), c_float(scale), _sink(None if sinks is not None else sink),
-        _ptr(sinks), c_int(1 if exact_weights else 0), _stream())
+        _ptr(sinks), c_int(1 if exact_weights else 0), c_float(softcap or 0.0), _stream())
 
 
 LATENT_TILES_PER_RANGE = 4      # a key range of the latent attention is at least this many tiles of 32 keys
@@ -303,11 +305,10 @@ TCGEN05_ATTENTION_MIN_TOKENS = 128     # shorter steps: the mma.sync kernel with
 
 
 def attention_prefill_tcgen05_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads: int, scale: float,
-                                   sink=None, exact_weights: bool = False) -> bool:
+                                   sink=None, exact_weights: bool = False, softcap=None) -> bool:
     """tcgen05 / TMA attention for steps with long runs of new tokens: one block per SM draws
-    items of 128 tokens of one head, scores and output in tensor memory.  ``exact_weights``: as
-    ``attention_prefill_bf16``.  A wait that ran out
-    shows in ``tc_status``."""
+    items of 128 tokens of one head, scores and output in tensor memory.  ``exact_weights``,
+    ``softcap``: as ``attention_prefill_bf16``.  A wait that ran out shows in ``tc_status``."""
     d = kv.head_dim
     if d not in (64, 128) or qkv.dtype != torch.bfloat16 or kv.k.dtype != torch.bfloat16:
         return False
@@ -318,7 +319,8 @@ def attention_prefill_tcgen05_bf16(ctx, qkv: torch.Tensor, out: torch.Tensor, kv
         _ptr(kv.k), _ptr(kv.v), c_long(kv.k.shape[0]), _ptr(kv.block_table), c_int(kv.block_table.stride(0)),
         _ptr(ctx.cu_seqlens), _ptr(ctx.seq_slot), _ptr(ctx.seq_start), c_int(ctx.n_seqs), c_long(qkv.shape[0]),
         c_int(ctx.max_seq_tokens), c_int(n_heads), c_int(kv.n_kv_heads), c_int(d), c_int(kv.window or 0),
-        c_int(kv.keep_first), c_float(scale), _sink(sink), c_int(1 if exact_weights else 0), _ptr(tc_status(qkv.device)), _stream())
+        c_int(kv.keep_first), c_float(scale), _sink(sink), c_int(1 if exact_weights else 0), c_float(softcap or 0.0),
+        _ptr(tc_status(qkv.device)), _stream())
 
 
 def attention_prefill_tcgen05_wait_probe(ctx, qkv: torch.Tensor, out: torch.Tensor, kv, n_heads: int, scale: float,
@@ -356,3 +358,24 @@ def lightning_chunks_bf16(proj: torch.Tensor, q_off: int, k_off: int, v_off: int
         "bfi_lightning_chunks_bf16", _ptr(proj), c_long(proj.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off),
         _ptr(out), c_long(out.stride(0)), _ptr(state), _ptr(decay), _ptr(cu_seqlens), _ptr(seq_slot), c_int(n_seqs),
         c_int(n_heads), c_int(dim), c_int(vdim), c_int(act), *rope, c_float(k_scale), _ptr(status), _stream())
+
+
+MLSTM_CHUNK_MIN_TOKENS = 8         # shorter runs of new tokens: the token-by-token kernel
+
+
+def mlstm_chunks_bf16(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: torch.Tensor, bias_i: torch.Tensor,
+                      bias_f: torch.Tensor, cap: float, q_scale: float, out: torch.Tensor, state: torch.Tensor, tails: torch.Tensor,
+                      cu_seqlens: torch.Tensor, seq_slot: torch.Tensor, n_seqs: int, n_heads: int, dim: int, vdim: int,
+                      columns: int = 0) -> bool:
+    """The matrix memory over runs of new tokens, 64 at a time on the tensor cores.  Same arguments and state as
+    ``ops.mlstm_scan``; False for sizes it does not take (head sizes that are no multiples of 16, or too large).
+    ``columns``: value columns per block (16, 32 or 64), for tests and measurements (0: the kernel's choice)."""
+    if proj.dtype != torch.bfloat16:
+        return False
+    check_memory(proj, q_off, k_off, v_off, bias_i, bias_f, out, state, tails, n_heads, dim, vdim, cu_seqlens, seq_slot)
+    check_memory_gates(gates, proj.shape[0], n_heads)
+    return library("fast").call_optional(
+        "bfi_mlstm_chunks_bf16", _ptr(proj), c_long(proj.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off), _ptr(gates),
+        c_long(gates.stride(0)), _ptr(bias_i), _ptr(bias_f), c_float(cap), c_float(q_scale), _ptr(out), c_long(out.stride(0)),
+        _ptr(state), _ptr(tails), _ptr(cu_seqlens), _ptr(seq_slot), c_int(n_seqs), c_int(n_heads), c_int(dim), c_int(vdim),
+        c_int(columns), _stream())

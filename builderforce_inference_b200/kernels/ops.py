@@ -77,19 +77,20 @@ def convert(src: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
 
 
 def embed_rows(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor,
-               status: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
-    """``out[t] = table[ids[t]] * scale`` into the float32 residual stream."""
+               status: Optional[torch.Tensor] = None, scale: float = 1.0, copies: int = 1) -> None:
+    """``out[t] = table[ids[t]] * scale`` into the float32 residual stream, ``copies`` times side by side."""
     _need_cuda(table, ids, out, status)
     _rows_2d(table, "embedding table")
     _rows_2d(out, "embedding output")
     _i32(ids, "token ids")
-    if out.dtype != torch.float32 or not out.is_contiguous() or out.shape != (ids.numel(), table.shape[1]):
-        raise KernelError("embedding output must be contiguous float32 [tokens, width]")
+    if out.dtype != torch.float32 or not out.is_contiguous() or copies < 1 \
+            or out.shape != (ids.numel(), copies * table.shape[1]):
+        raise KernelError("embedding output must be contiguous float32 [tokens, copies * width]")
     if not table.is_contiguous():
         raise KernelError("embedding table must be contiguous")
     library("core").call("bfi_embed_rows", _ptr(table), c_int(dtype_code(table.dtype)), _ptr(ids), _ptr(out),
-                         c_int(ids.numel()), c_int(table.shape[1]), c_int(table.shape[0]), c_float(scale), _ptr(status),
-                         _stream())
+                         c_int(ids.numel()), c_int(table.shape[1]), c_int(table.shape[0]), c_float(scale),
+                         c_int(copies), _ptr(status), _stream())
 
 
 def rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor,
@@ -325,11 +326,12 @@ def gated_rmsnorm(x: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: flo
 
 def attention_paged(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv, cu_seqlens: torch.Tensor,
                     seq_slot: torch.Tensor, seq_start: torch.Tensor, n_seqs: int, max_tokens: int,
-                    n_q: int, scale: float, sink=None) -> None:
+                    n_q: int, scale: float, sink=None, softcap: Optional[float] = None) -> None:
     """``q`` is the first query element of the step (a view into the qkv buffer); token ``t``, head
     ``h`` lies at ``q + t*q_stride + h*head_dim``.  ``out`` is ``[tokens, n_q*v_dim]``.  With
     ``sink`` (a number, or a float32 tensor with one per query head) the softmax's denominator
-    carries ``exp(sink)`` beside the keys' terms.  The cache view says whether the values have a
+    carries ``exp(sink)`` beside the keys' terms.  With ``softcap`` a score becomes ``softcap * tanh(score / softcap)``
+    before the softmax.  The cache view says whether the values have a
     size of their own (or are the first values of the keys) and whether a token reads only its own
     chunk of positions."""
     has_sink, sink_value, sinks = 0, 0.0, None
@@ -352,7 +354,8 @@ def attention_paged(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv, cu_se
         c_int(kv.block_table.stride(0)),
         _ptr(cu_seqlens), _ptr(seq_slot), _ptr(seq_start), c_int(n_seqs), c_int(max_tokens), c_int(n_q),
         c_int(kv.n_kv_heads), c_int(kv.head_dim), c_int(kv.value_dim), c_int(kv.window or 0), c_int(kv.keep_first),
-        c_int(kv.chunk or 0), c_float(scale), c_int(has_sink), c_float(sink_value), _ptr(sinks), _stream())
+        c_int(kv.chunk or 0), c_float(scale), c_int(has_sink), c_float(sink_value), _ptr(sinks),
+        c_float(softcap or 0.0), _stream())
 
 
 def latent_prepare(proj: torch.Tensor, qa: torch.Tensor, n_heads: int, dim: int, rot_dim: int, rank: int, kv_off: int,
@@ -922,6 +925,147 @@ def moe_weigh_dense(act: torch.Tensor, n_experts: int, idx: torch.Tensor, weight
     library("core").call("bfi_moe_weigh_dense", _ptr(act), c_long(act.stride(0)), c_int(dtype_code(act.dtype)), _ptr(idx),
                          _ptr(weight), _ptr(token_slot), c_int(n), c_int(top), c_int(n_experts), c_int(routed // n_experts),
                          c_int(tail), _ptr(gate), c_int(kind), _stream())
+
+
+def _norm_args(alpha, w, b, width: int, out, n: int, what: str) -> list:
+    """A dynamic tanh's arguments, checked: ``(alpha, w, b)`` and where it is written (None: no norm)."""
+    if alpha is None:
+        return [_ptr(None), _ptr(None), c_int(0), _ptr(None), c_int(0), _ptr(None), c_int(0), c_long(0)]
+    _f32_vector(alpha, 1, f"{what}: alpha")
+    for t in (w, b):
+        if t.shape != (width,) or not t.is_contiguous():
+            raise KernelError(f"{what}: weight and bias must be contiguous [{width}]")
+    _rows_2d(out, f"{what}: output")
+    if out.shape != (n, width):
+        raise KernelError(f"{what}: output must be [{n}, {width}], got {tuple(out.shape)}")
+    return [_ptr(alpha), _ptr(w), c_int(dtype_code(w.dtype)), _ptr(b), c_int(dtype_code(b.dtype)), _ptr(out),
+            c_int(dtype_code(out.dtype)), c_long(out.stride(0))]
+
+
+def dynamic_tanh(x: torch.Tensor, out: Optional[torch.Tensor], alpha: Optional[torch.Tensor], w: Optional[torch.Tensor],
+                 b: Optional[torch.Tensor], rows: Optional[torch.Tensor] = None, streams: int = 1,
+                 read: Optional[torch.Tensor] = None, u_out: Optional[torch.Tensor] = None) -> None:
+    """``out[r] = tanh(alpha * u) * w + b`` with ``u = x[rows[r]]`` (``rows`` None: every row in order), or, for
+    rows of ``streams`` copies, ``u = sum_a read[a] * x[rows[r], a]`` (``read`` None: the plain sum).  ``u_out``
+    (float32) receives ``u``; with ``alpha`` None that is all."""
+    _need_cuda(x, out, alpha, w, b, rows, read, u_out)
+    _rows_2d(x, "norm input")
+    _i32(rows, "row indices")
+    if x.dtype != torch.float32 or x.shape[1] % streams != 0:
+        raise KernelError("dynamic_tanh: the input must be float32 rows of whole copies")
+    width = x.shape[1] // streams
+    n = rows.numel() if rows is not None else x.shape[0]
+    _f32_vector(read, streams, "dynamic_tanh: the copies' weights")
+    if u_out is not None and (u_out.dtype != torch.float32 or u_out.shape != (n, width) or u_out.stride(1) != 1):
+        raise KernelError("dynamic_tanh: the sum must be float32 [rows, width]")
+    norm = _norm_args(alpha, w, b, width, out, n, "dynamic_tanh")
+    library("core").call("bfi_dynamic_tanh", _ptr(x), c_long(x.stride(0)), _ptr(rows), c_int(streams), _ptr(read), c_int(n),
+                         c_int(width), *norm, _ptr(u_out), c_long(0 if u_out is None else u_out.stride(0)), _stream())
+
+
+def stream_mix(x: torch.Tensor, streams: int, terms, scale: Optional[torch.Tensor], mix: torch.Tensor, write: torch.Tensor,
+               read: Optional[torch.Tensor] = None, norm=None, out: Optional[torch.Tensor] = None,
+               u_out: Optional[torch.Tensor] = None) -> None:
+    """A sublayer's output into the ``streams`` copies of the residual stream ``x`` (float32
+    ``[tokens, streams * width]``), all copies from the old ones: with ``y = scale * sum_i c_i y_i`` over the one or two
+    ``terms`` ``(y_i, c_i)`` (float32 ``[tokens, width]``; ``scale`` ``[width]`` or None),
+    ``x[t, b] = sum_a mix[a, b] * x[t, a] + write[b] * y[t]``.  With ``read`` what the next sublayer reads is made from the
+    new copies: ``u = sum_b read[b] * x[t, b]`` into ``u_out`` (float32) and / or, with ``norm`` ``(alpha, w, b)``,
+    its dynamic tanh into ``out``."""
+    tensors = [x, scale, mix, write, read, out, u_out] + [y for y, _ in terms]
+    _need_cuda(*tensors)
+    _rows_2d(x, "residual stream")
+    if x.dtype != torch.float32 or x.shape[1] % streams != 0 or not 1 <= len(terms) <= 2:
+        raise KernelError("stream_mix: float32 rows of whole copies, and one or two terms")
+    n, width = x.shape[0], x.shape[1] // streams
+    for y, _ in terms:
+        _rows_2d(y, "sublayer output")
+        if y.dtype != torch.float32 or y.shape != (n, width):
+            raise KernelError("stream_mix: a sublayer's output must be float32 [tokens, width]")
+    if scale is not None and (scale.shape != (width,) or not scale.is_contiguous()):
+        raise KernelError(f"stream_mix: the scale must be contiguous [{width}]")
+    _f32_vector(mix, streams * streams, "stream_mix: the matrix")
+    _f32_vector(write, streams, "stream_mix: the output's weights")
+    _f32_vector(read, streams, "stream_mix: the input's weights")
+    if (norm is not None or u_out is not None) and read is None:
+        raise KernelError("stream_mix: what the next sublayer reads needs its weights")
+    if u_out is not None and (u_out.dtype != torch.float32 or u_out.shape != (n, width) or u_out.stride(1) != 1):
+        raise KernelError("stream_mix: the next sublayer's sum must be float32 [tokens, width]")
+    alpha, w, b = norm if norm is not None else (None, None, None)
+    _need_cuda(alpha, w, b)
+    norm_args = _norm_args(alpha, w, b, width, out, n, "stream_mix")
+    (y0, c0), (y1, c1) = terms[0], (terms[1] if len(terms) == 2 else (None, 0.0))
+    library("core").call("bfi_stream_mix", _ptr(x), c_long(x.stride(0)), c_int(streams), c_int(n), c_int(width), _ptr(y0),
+                         c_long(y0.stride(0)), c_float(c0), _ptr(y1), c_long(0 if y1 is None else y1.stride(0)), c_float(c1),
+                         _ptr(scale), c_int(0 if scale is None else dtype_code(scale.dtype)), _ptr(mix), _ptr(write), _ptr(read),
+                         *norm_args, _ptr(u_out), c_long(0 if u_out is None else u_out.stride(0)), _stream())
+
+
+def check_memory(proj, q_off: int, k_off: int, v_off: int, bias_i, bias_f, out, state, tails, n_heads: int, dim: int, vdim: int,
+                 cu_seqlens, seq_slot) -> None:
+    """The arguments the matrix memory's kernels share."""
+    _need_cuda(proj, bias_i, bias_f, out, state, tails, cu_seqlens, seq_slot)
+    _rows_2d(proj, "projections")
+    _rows_2d(out, "recurrence output")
+    _i32(cu_seqlens, "cu_seqlens")
+    _i32(seq_slot, "sequence slots")
+    _f32_vector(bias_i, n_heads, "matrix memory: the input gate's bias")
+    _f32_vector(bias_f, n_heads, "matrix memory: the forget gate's bias")
+    if out.dtype != torch.float32 or out.shape != (proj.shape[0], n_heads * vdim):
+        raise KernelError("matrix memory: the output must be float32 [tokens, heads * vdim]")
+    if state.dtype != torch.float32 or not state.is_contiguous() or tuple(state.shape[1:]) != (n_heads, dim, vdim):
+        raise KernelError("matrix memory: the state must be contiguous float32 [slots, heads, dim, vdim]")
+    if tails.dtype != torch.float32 or not tails.is_contiguous() or tuple(tails.shape) != (state.shape[0], n_heads, dim + 2):
+        raise KernelError("matrix memory: the heads' tails must be contiguous float32 [slots, heads, dim + 2]")
+    if max(q_off, k_off) + n_heads * dim > proj.shape[1] or v_off + n_heads * vdim > proj.shape[1] or min(q_off, k_off, v_off) < 0:
+        raise KernelError("matrix memory: the projections' row is shorter than the heads")
+
+
+def check_memory_gates(gates, n_tokens: int, n_heads: int) -> None:
+    _need_cuda(gates)
+    _rows_2d(gates, "gate logits")
+    if gates.dtype != torch.float32 or gates.shape != (n_tokens, 2 * n_heads):
+        raise KernelError("matrix memory: the gates' logits must be float32 [tokens, 2 * heads]")
+
+
+def mlstm_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, gates: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor,
+               cap: float, q_scale: float, out: torch.Tensor, state: torch.Tensor, tails: torch.Tensor, cu_seqlens: torch.Tensor,
+               seq_slot: torch.Tensor, n_seqs: int, n_heads: int, dim: int, vdim: int) -> None:
+    """The matrix memory (mLSTM) over the step's new tokens, token by token.  q, k, v are columns ``q_off``,
+    ``k_off``, ``v_off`` of ``proj`` (q is multiplied by ``q_scale``); ``gates`` float32 ``[tokens, 2 * heads]`` holds
+    the logits of the input gates, then of the forget gates; with ``c(z) = cap * tanh(z / cap)``, ``i = c(z_i + b_i)``,
+    ``f = log sigmoid(c(z_f + b_f))``:
+
+        m' = max(f + m, i);  S = e^(f + m - m') S + e^(i - m') k v^T;  n likewise with k alone
+        o = S^T q / (max(|n . q|, e^-m') + 1e-6)
+
+    ``state`` float32 ``[slots, heads, dim, vdim]`` carries S, ``tails`` ``[slots, heads, dim + 2]`` n, m and a counter
+    that is zero between launches; ``out`` is float32 ``[tokens, heads * vdim]``."""
+    check_memory(proj, q_off, k_off, v_off, bias_i, bias_f, out, state, tails, n_heads, dim, vdim, cu_seqlens, seq_slot)
+    check_memory_gates(gates, proj.shape[0], n_heads)
+    library("core").call("bfi_mlstm_scan", _ptr(proj), c_int(dtype_code(proj.dtype)), c_long(proj.stride(0)), c_int(q_off), c_int(k_off),
+                         c_int(v_off), _ptr(gates), c_long(gates.stride(0)), _ptr(bias_i), _ptr(bias_f), c_float(cap), c_float(q_scale),
+                         _ptr(out), c_long(out.stride(0)), _ptr(state), _ptr(tails), _ptr(cu_seqlens), _ptr(seq_slot), c_int(n_seqs),
+                         c_int(n_heads), c_int(dim), c_int(vdim), _stream())
+
+
+def mlstm_step(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, x: torch.Tensor, w_gate: torch.Tensor, bias_i: torch.Tensor,
+               bias_f: torch.Tensor, cap: float, q_scale: float, out: torch.Tensor, state: torch.Tensor, tails: torch.Tensor,
+               cu_seqlens: torch.Tensor, seq_slot: torch.Tensor, n_seqs: int, n_heads: int, dim: int, vdim: int) -> bool:
+    """``mlstm_scan`` for steps in which every sequence brings exactly one token; the gates' logits are made in the
+    same kernel from ``x`` ``[tokens, width]`` and ``w_gate`` ``[2 * heads, width]`` (both of the projections' dtype).
+    False for heads of more than 256 key values."""
+    check_memory(proj, q_off, k_off, v_off, bias_i, bias_f, out, state, tails, n_heads, dim, vdim, cu_seqlens, seq_slot)
+    _need_cuda(x, w_gate)
+    _rows_2d(x, "gate input")
+    if x.dtype != proj.dtype or w_gate.dtype != proj.dtype or x.shape[0] != proj.shape[0] or not w_gate.is_contiguous() \
+            or w_gate.shape != (2 * n_heads, x.shape[1]):
+        raise KernelError("mlstm_step: input [tokens, width] and gate weights [2 * heads, width] of the projections' dtype")
+    return library("core").call_optional(
+        "bfi_mlstm_step", _ptr(proj), c_int(dtype_code(proj.dtype)), c_long(proj.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off),
+        _ptr(x), c_long(x.stride(0)), _ptr(w_gate), c_int(x.shape[1]), _ptr(bias_i), _ptr(bias_f), c_float(cap), c_float(q_scale),
+        _ptr(out), c_long(out.stride(0)), _ptr(state), _ptr(tails), _ptr(cu_seqlens), _ptr(seq_slot), c_int(n_seqs), c_int(n_heads),
+        c_int(dim), c_int(vdim), _stream())
 
 
 def gemm_simt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = EPI_STORE) -> None:

@@ -30,7 +30,8 @@ this layer, as they are cached, are also left in a buffer of the step; ``"mix"``
 ``(1 - lambda) v + lambda v_source`` with the source layer's values of the same token and a learned
 number ``lambda``, before they are cached; both ride on the convolution's kernel); ``gate``
 (``"head"``: head a's output is multiplied by ``sigmoid(W_g h)_a``, the logits coming out of the same
-product as q, k and v).  The plain
+product as q, k and v); ``softcap`` (a score becomes ``softcap * tanh(score / softcap)`` before the
+softmax, in every kernel as the scores leave the product).  The plain
 combination (no bias, head norm or none, own values, rotate-half) runs the per-head kernel that
 fuses norm, rotation and cache write; the others run the per-token kernel that also adds the
 biases, so no variant costs a launch of its own.
@@ -57,7 +58,7 @@ class Attention(Mixer):
                  bias: bool = False, values: str = "projection", sink=None, v_dim: Optional[int] = None,
                  chunk: Optional[int] = None, out_bias: Optional[bool] = None, exact_weights: bool = False,
                  conv_taps: Optional[int] = None, v_mix: Optional[str] = None, gate: Optional[str] = None,
-                 keep_first: int = 0):
+                 keep_first: int = 0, softcap: Optional[float] = None):
         if n_heads % n_kv_heads != 0:
             raise ValueError(f"GQA: {n_heads} query heads do not divide into {n_kv_heads} kv heads")
         if head_dim % 2 != 0 or head_dim > 512:
@@ -76,6 +77,9 @@ class Attention(Mixer):
             raise ValueError(f"chunk must be positive, got {chunk}")
         if keep_first < 0 or (keep_first > 0 and chunk is not None):
             raise ValueError(f"first positions are kept beside a window, not beside a chunk; got keep_first {keep_first}")
+        if softcap is not None and not softcap > 0:
+            raise ValueError(f"the cap on the scores must be positive, got {softcap}")
+        self.softcap = None if softcap is None else float(softcap)
         v_dim = head_dim if v_dim is None else int(v_dim)
         if v_dim < 1 or v_dim > 512:
             raise ValueError(f"attention kernels take value sizes from 1 to 512, got {v_dim}")
@@ -265,7 +269,7 @@ class Attention(Mixer):
     def attend(self, ctx, qkv, out, kv) -> None:
         from ..kernels import attention as fast_attention
         sink = self.sinks if self.learned_sink else self.sink
-        if fast_attention.attend(ctx, qkv, out, kv, self.n_heads, self.scale, sink, self.exact_weights):
+        if fast_attention.attend(ctx, qkv, out, kv, self.n_heads, self.scale, sink, self.exact_weights, self.softcap):
             return
         ops.attention_paged(qkv, qkv.stride(0), out, kv, ctx.cu_seqlens, ctx.seq_slot, ctx.seq_start,
-                            ctx.n_seqs, ctx.max_seq_tokens, self.n_heads, self.scale, sink)
+                            ctx.n_seqs, ctx.max_seq_tokens, self.n_heads, self.scale, sink, self.softcap)

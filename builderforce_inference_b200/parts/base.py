@@ -133,6 +133,17 @@ class Norm(Part):
     def forward(self, ctx, x, rows=None):
         raise NotImplementedError
 
+    def forward_streams(self, ctx, x, streams: int, read, rows=None, tag: str = "norm.out"):
+        """The norm of ``sum_a read[a] * x[:, a]`` over the ``streams`` copies in a row of ``x`` (``read`` float32,
+        None: the plain sum).  A norm whose kernel takes the sum along overrides this."""
+        import torch
+
+        from ..kernels import ops
+        n = x.shape[0] if rows is None else rows.numel()
+        u = ctx.rows("streams.sum", x.shape[1] // streams, torch.float32, n_rows=n)
+        ops.dynamic_tanh(x, None, None, None, None, rows=rows, streams=streams, read=read, u_out=u)
+        return self.forward(ctx, u, tag=tag)
+
 
 class InputPart(Part):
     """Something added to the residual stream right after the token embedding.  It may keep a
@@ -179,6 +190,14 @@ class Mixer(Part):
         product can store overrides this and saves the clearing."""
         out.zero_()
         self.forward(ctx, h, out, run)
+
+    def forward_terms(self, ctx, h, width: int, run) -> list:
+        """The mixer's output as one or two float32 buffers ``[tokens, width]`` with a factor each, for blocks
+        whose next kernel can take their sum along."""
+        import torch
+        y = ctx.rows("sublayer.out", width, torch.float32)
+        self.forward_store(ctx, h, y, run)
+        return [(y, 1.0)]
 
 
 class FeedForward(Part):
@@ -275,5 +294,6 @@ class ModelSpec:
     embedding_scale: float = 1.0       # the embedding rows are multiplied by it; the tied head is not
     logit_scale: float = 1.0           # the logits are multiplied by it
     logit_softcap: Optional[float] = None   # c: the logits become c * tanh(logits / c)
+    streams: int = 1                   # copies of the residual stream, side by side in a token's row; the logits see their sum
     # parts added to the embedded tokens, each with the checkpoint names of its tensors: (PartSpec, names)
     input_parts: Sequence[Tuple[PartSpec, Mapping[str, str]]] = ()

@@ -24,6 +24,14 @@ the mixer's and the feed-forward's last matrix product.
               convolution, of this block or of the out-norm block that runs next) from the row it has
               just written, so a sublayer costs one launch around it instead of two.  The feed-forward
               (with its norm, convolution and gate) may be absent.
+``hyper``     the residual stream is held ``streams`` times (a token's copies side by side in its row).
+              Sublayer i reads ``u = sum_a read_i[a] X_a`` through its norm; with ``y = scale_i * sublayer(norm_i(u))``
+              (``scale_i``, a factor per channel, with ``layer_scale``) all copies are renewed from the old
+              ones: ``X_b <- sum_a mix_i[a, b] X_a + write_i[b] y``.  One kernel scales, mixes and writes and
+              also makes what the next sublayer reads (of this block or of the hyper block that runs
+              next) from the copies it has in registers: its norm's output where that norm computes no
+              statistics (``dynamic_tanh``), the sum ``u`` otherwise.  A mixer that is a weighted sum hands its
+              members' outputs over unsummed.  The feed-forward may be absent.
 """
 from __future__ import annotations
 
@@ -33,6 +41,7 @@ from ..cache.cache import KVView, RunCache, needs_of
 from ..kernels import ops
 from ..kernels.linear import EPI_STORE, linear
 from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, ParamSpec, PartSpec, StateNeed
+from .norm import DynamicTanh
 
 
 @BLOCKS.register("prenorm")
@@ -263,3 +272,86 @@ class OutNormBlock(Block):
             made = self._output(ctx, residual, y, plain, 1, self.norm2, follow=to_next)
         if to_next is not None:
             ctx.extras["outnorm.input"] = (after, made)
+
+
+@BLOCKS.register("hyper")
+class HyperBlock(Block):
+    graph_safe = True
+
+    def __init__(self, width: int, streams: int, norm1: PartSpec, mixer: PartSpec, norm2: PartSpec = None, ffn: PartSpec = None,
+                 layer_scale: bool = False):
+        if (ffn is None) != (norm2 is None):
+            raise ValueError("a hyper block has a feed-forward with its norm, or neither")
+        if not 1 <= streams <= 32:
+            raise ValueError(f"a hyper block holds the residual stream 1 to 32 times, got {streams}")
+        self.width, self.streams, self.layer_scale = int(width), int(streams), bool(layer_scale)
+        self.norms = [NORMS.build(norm1)] + ([NORMS.build(norm2)] if ffn is not None else [])
+        self._mixer = MIXERS.build(mixer)
+        self.ffn = FEED_FORWARDS.build(ffn) if ffn is not None else None
+        self.n_sub = len(self.norms)
+        self.read, self.write, self.mix, self.scale = ([None] * self.n_sub for _ in range(4))
+
+    def children(self):
+        out = {"norm1": self.norms[0], "mixer": self._mixer}
+        if self.ffn is not None:
+            out.update({"norm2": self.norms[1], "ffn": self.ffn})
+        return out
+
+    def mixer(self):
+        return self._mixer
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        specs = {}
+        for i in range(1, self.n_sub + 1):
+            specs.update({f"read{i}": ParamSpec((self.streams,), "norm"), f"write{i}": ParamSpec((self.streams,), "norm"),
+                          f"mix{i}": ParamSpec((self.streams, self.streams))})
+            if self.layer_scale:
+                specs[f"scale{i}"] = ParamSpec((self.width,), "norm")
+        return specs
+
+    def load(self, tensors, runtime) -> None:
+        for i in range(self.n_sub):
+            for name in ("read", "write", "mix"):
+                getattr(self, name)[i] = tensors[f"{name}{i + 1}"].float().contiguous()
+            if self.layer_scale:
+                self.scale[i] = tensors[f"scale{i + 1}"].contiguous()
+
+    def _input(self, ctx, x, i: int):
+        return self.norms[i].forward_streams(ctx, x, self.streams, self.read[i])
+
+    def _renew(self, ctx, x, i: int, terms, then: "HyperBlock", j: int):
+        """Sublayer ``i``'s output into the copies.  Returns the input of sublayer ``j`` of ``then`` (None: nothing
+        follows that this kernel could make)."""
+        if then is None:
+            ops.stream_mix(x, self.streams, terms, self.scale[i], self.mix[i], self.write[i])
+            return None
+        norm = then.norms[j]
+        if isinstance(norm, DynamicTanh):
+            h = ctx.rows("norm.out", self.width)
+            ops.stream_mix(x, self.streams, terms, self.scale[i], self.mix[i], self.write[i], read=then.read[j], norm=norm.args, out=h)
+            return h
+        import torch
+        u = ctx.rows("streams.sum", self.width, torch.float32)
+        ops.stream_mix(x, self.streams, terms, self.scale[i], self.mix[i], self.write[i], read=then.read[j], u_out=u)
+        return norm.forward(ctx, u)
+
+    def forward(self, ctx, residual, run) -> None:
+        import torch
+        if residual.shape[1] != self.streams * self.width:
+            raise RuntimeError(f"a hyper block of {self.streams} copies got rows of {residual.shape[1]} values")
+        after = ctx.extras.get("next_block")
+        if not (isinstance(after, HyperBlock) and (after.width, after.streams) == (self.width, self.streams)):
+            after = None
+        # the kernel before may have made this block's first input (a looped block may follow itself)
+        made = ctx.extras.pop("hyper.input", None)
+        h = made[1] if made is not None and made[0] is self else self._input(ctx, residual, 0)
+        terms = self._mixer.forward_terms(ctx, h, self.width, run)
+        if self.ffn is None:
+            h = self._renew(ctx, residual, 0, terms, after, 0)
+        else:
+            h = self._renew(ctx, residual, 0, terms, self, 1)
+            y = ctx.rows("sublayer.out", self.width, torch.float32)
+            self.ffn.forward_store(ctx, h, y)
+            h = self._renew(ctx, residual, 1, [(y, 1.0)], after, 0)
+        if after is not None:
+            ctx.extras["hyper.input"] = (after, h)

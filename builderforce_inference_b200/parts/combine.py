@@ -1,7 +1,7 @@
 """A mixer that is the weighted sum of several mixers reading the same input:
 ``out = sum_i scale_i * mixer_i(h)``.  Every member keeps the cache it asks for (the run's cache
 then carries the members' needs one after the other) and writes its output to a float32 buffer of
-its own; the sum is taken in float32.
+its own; the sum is taken in float32, by a kernel of its own or by the block's (``forward_terms``).
 """
 from __future__ import annotations
 
@@ -54,15 +54,18 @@ class WeightedSumMixer(Mixer):
             out.append(RunCache(kv=kv, state=state, writes_cache=run.writes_cache, entries=entries))
         return out
 
-    def forward_store(self, ctx, h, out, run) -> None:
+    def forward_terms(self, ctx, h, width, run):
         runs = self._member_runs(run)
-        parts = []
+        terms = []
         for i, n in enumerate(self.names):
-            y = ctx.rows(f"sum.member{i}", out.shape[1], torch.float32)
+            y = ctx.rows(f"sum.member{i}", width, torch.float32)
             self.members[n].forward_store(ctx, h, y, runs[i])
-            parts.append(y)
-        a, b = (self.scales[n] for n in self.names)
-        ops.weighted_sum(out, parts[0], a, parts[1], b)
+            terms.append((y, self.scales[n]))
+        return terms
+
+    def forward_store(self, ctx, h, out, run) -> None:
+        (y0, a), (y1, b) = self.forward_terms(ctx, h, out.shape[1], run)
+        ops.weighted_sum(out, y0, a, y1, b)
 
     def forward(self, ctx, h, residual, run) -> None:
         y = ctx.rows("sum.out", residual.shape[1], torch.float32)

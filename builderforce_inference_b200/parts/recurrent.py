@@ -32,6 +32,15 @@ head's output is normed over ``vdim`` (one weight of ``vdim`` values for all hea
 where ``cand(u) = u + 1/2`` for ``u >= 0`` and ``sigmoid(u)`` below (``candidate="positive"``), or ``u``
 itself (``"identity"``).  Its gates read the current token only, so the recurrence is linear in S
 and the kernel cuts a sequence's tokens into segments that run side by side.
+
+``mlstm`` (the matrix memory of xLSTM) puts a normaliser beside the matrix and takes the gates as
+exponentials, kept in range by a running maximum (``kernels/ops.mlstm_scan``).  ``q = W_q h * dim^(-1/2)``,
+``k = W_k h``, ``v = W_v h``; per head a log input gate ``i = c(W_i h + b_i)`` and a log forget gate
+``f = log sigmoid(c(W_f h + b_f))`` with the soft cap ``c(z) = cap tanh(z / cap)``.  Every head's output is
+divided by its root mean square, multiplied by ``norm`` (a weight over all heads) and by ``sigmoid(W_g h)``,
+and projected.  The gates' logits are float32: a product of their own with a float32 result in steps
+with longer pieces, part of the recurrence's kernel in single-token steps.  A sequence keeps the matrix, the
+normaliser and the maximum of every head.
 """
 from __future__ import annotations
 
@@ -248,3 +257,85 @@ class MinGRU(Mixer):
         ops.gated_scan(proj, 0, n, 2 * n, n, self.b_z, self.b_x, y, state, ctx.cu_seqlens, ctx.seq_slot, ctx.n_seqs,
                        ctx.max_seq_tokens, cand=self.cand)
         linear(y, self.w_o, target, epilogue)
+
+
+@MIXERS.register("mlstm")
+class MatrixMemory(Mixer):
+    graph_safe = True
+
+    def __init__(self, width: int, n_heads: int, dim: int, vdim: int, gate_cap: float, eps: float = 1e-6):
+        if n_heads < 1 or dim < 1 or vdim < 1:
+            raise ValueError(f"matrix memory: bad sizes heads={n_heads} dim={dim} vdim={vdim}")
+        if not gate_cap > 0:
+            raise ValueError(f"matrix memory: the gates' cap must be positive, got {gate_cap}")
+        self.width, self.n_heads, self.dim, self.vdim = int(width), int(n_heads), int(dim), int(vdim)
+        self.cap, self.eps = float(gate_cap), float(eps)
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        qk, vv, w, h = self.n_heads * self.dim, self.n_heads * self.vdim, self.width, self.n_heads
+        return {"q_proj": ParamSpec((qk, w)), "k_proj": ParamSpec((qk, w)), "v_proj": ParamSpec((vv, w)), "g_proj": ParamSpec((vv, w)),
+                "i_proj": ParamSpec((h, w)), "i_proj.bias": ParamSpec((h,)), "f_proj": ParamSpec((h, w)), "f_proj.bias": ParamSpec((h,)),
+                "norm": ParamSpec((vv,), "norm"), "o_proj": ParamSpec((w, vv))}
+
+    def cache_need(self):
+        # n, m and the kernels' counter ride behind one another: dim + 2 values a head
+        return (StateNeed((self.n_heads, self.dim, self.vdim), "float32"), StateNeed((self.n_heads, self.dim + 2), "float32"))
+
+    def load(self, tensors, runtime) -> None:
+        # one product gives q, k, v and the output gate, every part starting on 16 bytes
+        parts, at, offs = [], 0, []
+        for name in ("q_proj", "k_proj", "v_proj", "g_proj"):
+            m = tensors[name]
+            if at % 8:
+                parts.append(torch.zeros(((-at) % 8, self.width), dtype=m.dtype, device=m.device))
+                at += (-at) % 8
+            offs.append(at)
+            parts.append(m)
+            at += m.shape[0]
+        if at % 8:
+            parts.append(torch.zeros(((-at) % 8, self.width), dtype=parts[0].dtype, device=parts[0].device))
+            at += (-at) % 8
+        if len({m.dtype for m in parts}) > 1:
+            parts = [m.float() for m in parts]
+        self.q_off, self.k_off, self.v_off, self.g_off = offs
+        self.w_in = torch.cat(parts, dim=0).contiguous()
+        gates = [tensors["i_proj"], tensors["f_proj"]]
+        if len({m.dtype for m in gates} | {self.w_in.dtype}) > 1:
+            gates = [m.float() for m in gates]
+        self.w_gate = torch.cat(gates, dim=0).contiguous()
+        self.bias_i, self.bias_f = _as_f32(tensors["i_proj.bias"]), _as_f32(tensors["f_proj.bias"])
+        self.norm, self.w_o = tensors["norm"].contiguous(), tensors["o_proj"]
+
+    def forward(self, ctx, h, residual, run) -> None:
+        self._run(ctx, h, residual, run, EPI_ACCUMULATE)
+
+    def forward_store(self, ctx, h, out, run) -> None:
+        self._run(ctx, h, out, run, EPI_STORE)
+
+    def _run(self, ctx, h, target, run, epilogue) -> None:
+        if not run.writes_cache or len(run.entries) < 2:
+            raise RuntimeError("a matrix memory needs a state of its own for its run")
+        vv = self.n_heads * self.vdim
+        proj = ctx.rows("mem.proj", self.w_in.shape[0])
+        linear(h, self.w_in, proj, EPI_STORE)
+        o = ctx.rows("mem.o", vv, torch.float32)
+        self.recur(ctx, h, proj, o, run.entries[0], run.entries[1])
+        y = ctx.rows("mem.y", vv)
+        ops.gated_group_norm(o, proj[:, self.g_off:self.g_off + vv], self.norm, self.eps, y, self.n_heads, gate_first=False,
+                             gate_act=ops.GATE_SIGMOID)
+        linear(y, self.w_o, target, epilogue)
+
+    def recur(self, ctx, h, proj, o, state, tails) -> None:
+        args = (self.bias_i, self.bias_f, self.cap, self.dim ** -0.5, o, state, tails, ctx.cu_seqlens, ctx.seq_slot, ctx.n_seqs,
+                self.n_heads, self.dim, self.vdim)
+        offs = (self.q_off, self.k_off, self.v_off)
+        if ctx.max_seq_tokens == 1 and ctx.n_tokens == ctx.n_seqs and self.w_gate.dtype == proj.dtype \
+                and ops.mlstm_step(proj, *offs, h, self.w_gate, *args):
+            return
+        gates = ctx.rows("mem.gates", 2 * self.n_heads, torch.float32)
+        linear(h, self.w_gate, gates, EPI_STORE)
+        if proj.dtype == torch.bfloat16:
+            from ..kernels import fast_ops
+            if ctx.max_seq_tokens >= fast_ops.MLSTM_CHUNK_MIN_TOKENS and fast_ops.mlstm_chunks_bf16(proj, *offs, gates, *args):
+                return
+        ops.mlstm_scan(proj, *offs, gates, *args)

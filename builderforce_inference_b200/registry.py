@@ -2,7 +2,7 @@
 
 A config.json names its architecture under ``architectures[0]`` (a class name such as
 ``Qwen3ForCausalLM``), ``model_type`` (``qwen3``) or ``architecture`` (``Datasun``, ``Bepilorn``, ``Munerax``, ``Kikelorn``,
-``Zirivik``).  Any of them selects the entry; the lookup is exact and case-sensitive, and an unknown name is answered with the list of known ones, as in
+``Zirivik``, ``Zitezen``).  Any of them selects the entry; the lookup is exact and case-sensitive, and an unknown name is answered with the list of known ones, as in
 the reference (crates/bfi-models/src/arch.rs:70-91).
 """
 from __future__ import annotations
@@ -86,6 +86,10 @@ def _register_builtin() -> None:
     from .config.zirivik import ZirivikConfig
     register_architecture(("Zirivik", "zirivik"),
                           Architecture(name="zirivik", config_class=ZirivikConfig, describe=zirivik.describe))
+    from .architectures import zitezen
+    from .config.zitezen import ZitezenConfig
+    register_architecture(("Zitezen", "zitezen"),
+                          Architecture(name="zitezen", config_class=ZitezenConfig, describe=zitezen.describe))
 
 
 _register_builtin()
