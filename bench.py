@@ -28,7 +28,9 @@ of every kernel of a prompt step and of a single-token step.  ``--design munerax
 query latent, a minGRU and chunked attention again, in out-norm blocks) beside the designs closest
 to them and Qwen3, and ``--design zirivik`` for Zirivik (two retention layers, an attention layer with a
 window and kept first tokens, and one that reads its keys; dense and routed feed-forwards in turn)
-beside Bepilorn, Datasun and Qwen3.
+beside Bepilorn, Datasun and Qwen3, and ``--design zitezen`` for Zitezen (four copies of the residual
+stream; two matrix-memory layers, latent attention with a query latent, and soft-capped attention with
+a matrix memory beside it; dense feed-forwards) beside Zirivik, Kikelorn and Qwen3.
 
 The work is one GPU's: for ``--gpus`` above 1 it says so and exits with 2.  The reference arm
 (``--impl reference``) is unavailable: the reference is a Rust workspace, there is no Rust
@@ -214,7 +216,7 @@ def prefill_flops(c, layers, lens):
 
 
 KERNEL_CLASSES = (("products", ("gemm", "skinny")), ("attention", ("attention",)),
-                  ("recurrence", ("lightning", "decay_scan", "causal_conv")), ("experts", ("moe_",)))
+                  ("recurrence", ("lightning", "decay_scan", "causal_conv", "mlstm")), ("experts", ("moe_",)))
 
 
 def prefill_breakdown(eng, step, by_kernel=False):
@@ -426,6 +428,27 @@ def zirivik_config(width, heads, kv, d, ff, layers):
             "logit_softcap": 50.0, "layers": out}
 
 
+ZITEZEN_STREAMS = 4            # copies of the residual stream in the design runs
+ZITEZEN_CAP = 50.0             # cap on the attention layers' scores; the memories' gates are capped at 15
+
+
+def zitezen_config(width, heads, kv, d, ff, layers):
+    """A Zitezen model of these layer sizes: of every four layers two are matrix memories (heads of the
+    attention's sizes), the third is latent attention as Kikelorn's in these runs (a cache row of
+    512 + d/2 values, a query latent of 3/8 of the width), the fourth soft-capped attention beside a
+    matrix memory of half the heads; a dense feed-forward in every layer."""
+    half = d // 2
+    mem = {"heads": heads, "dim": d, "vdim": d, "gate_cap": 15.0}
+    lat = {"heads": heads, "dim": half, "rot_dim": half, "vdim": d, "kv_rank": MUNERAX_LATENT, "q_rank": 3 * width // 8,
+           "scale": d ** -0.5, "rot": {"base": 1e6, "dims": half}}
+    pair = {"left": {"heads": heads, "kv_heads": kv, "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": ZITEZEN_CAP,
+                     "rot": {"base": 1e6, "dims": half}}, "left_scale": 0.5,
+            "right": dict(mem, heads=heads // 2), "right_scale": 1.0}
+    kinds = [("mlstm", mem), ("mlstm", mem), ("latent_attention", lat), ("parallel", pair)]
+    return {"architecture": "Zitezen", "vocab": DESIGN_VOCAB, "width": width, "streams": ZITEZEN_STREAMS, "norm": {"eps": 1e-6}, "loop": None,
+            "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
 def decode_breakdown(model, batch, ctx_len):
     """One instrumented single-token step (no graph, an event around every kernel) behind prompts of
     ``ctx_len`` tokens: milliseconds by kernel."""
@@ -459,7 +482,11 @@ def design_run(a) -> int:
         width, heads, kv, d, ff = DESIGN_SIZES[name]
         qwen3 = dict(CONFIG_4B, num_hidden_layers=layers, hidden_size=width, num_attention_heads=heads,
                      num_key_value_heads=kv, head_dim=d, intermediate_size=ff, vocab_size=DESIGN_VOCAB)
-        if a.design == "zirivik":       # beside the design with the same block and a routed feed-forward, the one with the same recurrence and windows, and the dense one
+        if a.design == "zitezen":       # beside the design with a matrix state per head, the one with the same latent attention, and the dense one
+            configs = {"zitezen": zitezen_config(width, heads, kv, d, ff, layers),
+                       "zirivik": zirivik_config(width, heads, kv, d, ff, layers),
+                       "kikelorn": kikelorn_config(width, heads, kv, d, ff, layers), "qwen3": qwen3}
+        elif a.design == "zirivik":     # beside the design with the same block and a routed feed-forward, the one with the same recurrence and windows, and the dense one
             configs = {"zirivik": zirivik_config(width, heads, kv, d, ff, layers),
                        "bepilorn": bepilorn_config(width, heads, kv, d, ff, layers),
                        "datasun": datasun_config(width, heads, kv, d, ff, layers), "qwen3": qwen3}
@@ -479,7 +506,7 @@ def design_run(a) -> int:
             configs = {k: v for k, v in configs.items() if k in a.only.split(",")}
         for design, cfg in configs.items():
             model = Model.from_random(cfg, seed=0, dtype="bfloat16", max_tokens=64 * 2048, max_seq_len=CONTEXT, max_batch=64)
-            by_kernel = a.design in ("bepilorn", "munerax", "kikelorn", "zirivik")
+            by_kernel = a.design in ("bepilorn", "munerax", "kikelorn", "zirivik", "zitezen")
             pf = prefill_run(model, PREFILL_TOKENS, 5, layers, breakdown=True, by_kernel=by_kernel)
             row = {"prefill_2048": {"ms": round(pf["ms"], 3), "tok_s": round(pf["tok_s"], 1), "breakdown": pf["breakdown"]}}
             for b in (8, 64):
@@ -501,9 +528,13 @@ def design_run(a) -> int:
                            "minGRU, chunked attention; out-norm blocks with %d taps in front of every sublayer and a gate behind it; "
                            "dense feed-forward with biases" % (DESIGN_WINDOW, KIKELORN_TAPS, MUNERAX_LATENT, KIKELORN_TAPS),
                "zirivik": "retention x2, attention (window %d and the first %d tokens) x1 and one that reads its keys; dense feed-forward "
-                          "in even layers, %d experts, 4 used, in odd ones" % (DESIGN_WINDOW, ZIRIVIK_KEEP, BEPILORN_EXPERTS)}[a.design]
+                          "in even layers, %d experts, 4 used, in odd ones" % (DESIGN_WINDOW, ZIRIVIK_KEEP, BEPILORN_EXPERTS),
+               "zitezen": "%d copies of the residual stream; matrix memory x2, latent attention (cache row %d + head/2, query latent) x1, "
+                          "attention (scores capped at %g) + matrix memory x1; dense feed-forward"
+                          % (ZITEZEN_STREAMS, MUNERAX_LATENT, ZITEZEN_CAP)}[a.design]
     beside = {"bepilorn": "datasun and qwen3", "munerax": "bepilorn and qwen3",
-              "kikelorn": "munerax, bepilorn and qwen3", "zirivik": "bepilorn, datasun and qwen3"}.get(a.design, "qwen3")
+              "kikelorn": "munerax, bepilorn and qwen3", "zirivik": "bepilorn, datasun and qwen3",
+              "zitezen": "zirivik, kikelorn and qwen3"}.get(a.design, "qwen3")
     print(json.dumps({"workloads": a.design + " beside " + beside
                       + " at equal layer sizes, builder-run beside the benchmark", "dtype": "bf16",
                       "layers": layers, "pattern": pattern, "vocab": DESIGN_VOCAB,
@@ -526,7 +557,10 @@ def kernel_run(a) -> int:
     --heads H`` (the latent attention; --rows 1: single tokens behind C cached ones), ``--kernel weight_stream --shape S [--stages R] [--ksplit Z]`` (the
     matrix read once through the few-row products' TMA rings and nothing else: the floor under
     them), ``--kernel causal_conv|gated_scan|norm_add_gated|bias_gelu --seqs N --rows T --width W`` (what stands in front
-    of and behind an out-norm block's sublayers, the minGRU's recurrence, the dense feed-forward's bias and GELU).
+    of and behind an out-norm block's sublayers, the minGRU's recurrence, the dense feed-forward's bias and GELU),
+    ``--kernel mlstm_chunks --seqs N --rows T`` / ``--kernel mlstm_step --rows B`` (the matrix memory over prompts / over
+    single tokens), ``--kernel stream_mix --rows T --width W`` (a sublayer's output into four copies of the residual
+    stream, and the next sublayer's dynamic tanh).  ``--softcap C``: the attention kernels with their scores capped.
     Weights rotate over enough copies to exceed L2.  Prints one JSON line."""
     import torch
     from builderforce_inference_b200.kernels import fast_ops
@@ -595,6 +629,49 @@ def kernel_run(a) -> int:
         # per token and head: scores and their use within a chunk (causal half of 64 x 64), q S and the state update
         flops = n_seq * t_new * h * (2.0 * d * d * 2 + (2.0 * 32 * (d + d) if chunks else 0.0))
         what = {"seqs": n_seq, "new_tokens": t_new, "heads": h, "dim": d, "vdim": d, "rotate": bool(a.rotate)}
+    elif a.kernel in ("mlstm_chunks", "mlstm_step"):
+        # the matrix memory: --seqs prompts of --rows tokens (chunks), or --rows sequences of one token (step)
+        from builderforce_inference_b200.kernels import ops
+        c = CONFIG_4B
+        h, d, w = c["num_attention_heads"], c["head_dim"], c["hidden_size"]
+        chunks = a.kernel == "mlstm_chunks"
+        n_seq, t_new = (a.seqs, a.rows) if chunks else (a.rows, 1)
+        n = n_seq * t_new
+        copies = 1 if chunks else max(2, int(400e6 // (n_seq * h * d * d * 4)) + 1)
+        proj = torch.randn(n, 4 * h * d, device=dev, dtype=torch.bfloat16)
+        o = torch.empty(n, h * d, device=dev)
+        states = [(torch.zeros(n_seq, h, d, d, device=dev), torch.zeros(n_seq, h, d + 2, device=dev)) for _ in range(copies)]
+        bias_i, bias_f = torch.full((h,), -1.0, device=dev), torch.linspace(2.0, 6.0, h, device=dev)
+        cu = torch.arange(0, (n_seq + 1) * t_new, t_new, dtype=torch.int32, device=dev)
+        slots = torch.arange(n_seq, dtype=torch.int32, device=dev)
+        gates = torch.randn(n, 2 * h, device=dev)
+        x, wg = torch.randn(n, w, device=dev, dtype=torch.bfloat16), torch.randn(2 * h, w, device=dev, dtype=torch.bfloat16) * 0.02
+
+        def one(i):
+            tail = (bias_i, bias_f, 15.0, d ** -0.5, o) + states[i % copies] + (cu, slots, n_seq, h, d, d)
+            if not (fast_ops.mlstm_chunks_bf16(proj, 0, h * d, 2 * h * d, gates, *tail) if chunks else
+                    ops.mlstm_step(proj, 0, h * d, 2 * h * d, x, wg, *tail)):
+                raise SystemExit(f"{a.kernel} does not take this shape")
+        bytes_moved = n_seq * h * (d * d + d + 1) * 4 * 2 + n * (3 * h * d * 2 + h * d * 4) + (n * 2 * h * 4 if chunks else n * w * 2)
+        flops = n * h * (2.0 * d * d * 2 + (2.0 * 32 * (d + d) if chunks else 0.0))
+        what = {"seqs": n_seq, "new_tokens": t_new, "heads": h, "dim": d, "vdim": d}
+    elif a.kernel == "stream_mix":
+        # one sublayer's output into four copies of the residual stream, and the next sublayer's dynamic tanh
+        from builderforce_inference_b200.kernels import ops
+        n, w, s = a.rows * a.seqs, a.width, ZITEZEN_STREAMS
+        copies = max(2, int(400e6 // (n * w * (s + 1) * 4)) + 1)
+        xs = [torch.randn(n, s * w, device=dev) for _ in range(copies)]
+        ys = [torch.randn(n, w, device=dev) for _ in range(copies)]
+        h = torch.empty(n, w, device=dev, dtype=torch.bfloat16)
+        scale, nw, nb = (torch.ones(w, device=dev, dtype=torch.bfloat16) for _ in range(3))
+        mix = torch.eye(s, device=dev) * 0.8 + 0.05
+        wr, rd, alpha = torch.ones(s, device=dev), torch.full((s,), 1.0 / s, device=dev), torch.full((1,), 0.5, device=dev)
+
+        def one(i):
+            ops.stream_mix(xs[i % copies], s, [(ys[i % copies], 1.0)], scale, mix, wr, read=rd, norm=(alpha, nw, nb), out=h)
+        bytes_moved = n * w * (2 * s * 4 + 4 + 2)
+        flops = 0.0
+        what = {"tokens": n, "width": w, "streams": s}
     elif a.kernel in ("causal_conv", "gated_scan", "norm_add_gated", "bias_gelu"):
         # the kernels around an out-norm block's sublayers and of the minGRU: --seqs prompts of --rows tokens, --width channels
         from builderforce_inference_b200.kernels import ops
@@ -800,7 +877,7 @@ def kernel_run(a) -> int:
         fn = {"attention_decode": fast_ops.attention_decode_bf16, "attention_prefill": fast_ops.attention_prefill_bf16,
               "attention_prefill_tcgen05": fast_ops.attention_prefill_tcgen05_bf16}[a.kernel]
         def one(i):
-            if not fn(ctx, q, out, kvs[i % copies], nq, d ** -0.5, exact_weights=a.exact_weights):
+            if not fn(ctx, q, out, kvs[i % copies], nq, d ** -0.5, exact_weights=a.exact_weights, softcap=a.softcap or None):
                 raise SystemExit(f"{a.kernel} does not take this shape")
 
         def visible(pos):               # keys the token at pos reads
@@ -811,7 +888,7 @@ def kernel_run(a) -> int:
             bytes_moved += n_seq * t_new * nq * d * 2 * 2          # q in, the heads' outputs out
         flops = 4.0 * nq * d * n_seq * sum(visible(p) for p in range(ctx_len - t_new, ctx_len))
         what = {"seqs": n_seq, "new_tokens": t_new, "context": ctx_len, "q_heads": nq, "kv_heads": nkv, "head_dim": d,
-                "window": a.window, "keep_first": a.keep_first, "exact_weights": bool(a.exact_weights)}
+                "window": a.window, "keep_first": a.keep_first, "exact_weights": bool(a.exact_weights), "softcap": a.softcap}
     for i in range(3):
         one(i)
     torch.cuda.synchronize()
@@ -945,7 +1022,7 @@ def main() -> int:
     ap.add_argument("--kernel", default=None, choices=["skinny_gemm", "gemm_tcgen05", "weight_stream", "qk_norm_rope", "attention_decode",
                                                        "attention_prefill", "attention_prefill_tcgen05", "lightning_chunks", "lightning_scan",
                                                        "qk_prepare", "decay_scan", "decay_step", "attention_latent", "causal_conv",
-                                                       "gated_scan", "norm_add_gated", "bias_gelu"],
+                                                       "gated_scan", "norm_add_gated", "bias_gelu", "mlstm_chunks", "mlstm_step", "stream_mix"],
                     help="time one kernel instead of the model (see kernel_run)")
     ap.add_argument("--width", type=int, default=2048, help="kernel mode, the channel-wise kernels: channels of a row")
     ap.add_argument("--shape", default="qkv", choices=sorted(KERNEL_SHAPES))
@@ -963,13 +1040,14 @@ def main() -> int:
     ap.add_argument("--layers", type=int, default=None, help="run fewer layers of the same sizes")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 points and the prefill")
-    ap.add_argument("--design", default=None, choices=["datasun", "bepilorn", "munerax", "kikelorn", "zirivik"],
+    ap.add_argument("--design", default=None, choices=["datasun", "bepilorn", "munerax", "kikelorn", "zirivik", "zitezen"],
                     help="instead of the benchmark: this design beside qwen3 at equal layer sizes (see design_run)")
     ap.add_argument("--sizes", default=None, help="with --design: names of DESIGN_SIZES, comma-separated (default: all)")
     ap.add_argument("--only", default=None, help="with --design: the designs to run, comma-separated (default: all of that run)")
     ap.add_argument("--window", type=int, default=0, help="kernel mode, attention: the last --window positions")
     ap.add_argument("--keep-first", type=int, default=0, help="kernel mode, attention: and the first --keep-first positions")
     ap.add_argument("--exact-weights", action="store_true", help="kernel mode, attention: weights float32 in effect")
+    ap.add_argument("--softcap", type=float, default=0.0, help="kernel mode, attention: scores capped softly at this size")
     ap.add_argument("--rotate", action="store_true", help="kernel mode, lightning: retention (rotated q and k, no activations)")
     a = ap.parse_args()
     if a.impl == "reference":
