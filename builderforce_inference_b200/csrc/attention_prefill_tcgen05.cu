@@ -543,7 +543,21 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 tmem_wait_ld();
                 if (CAP) {
 #pragma unroll
-                    for (int e = 0; e < FT_KEYS; ++e) s[e] = score_capped(s[e], cap);
+                    for (int c = 0; c < FT_KEYS / 32; ++c) {          // 32 keys at a time: scores near zero need no special functions
+                        float top = 0.0f;
+#pragma unroll
+                        for (int e = c * 32; e < c * 32 + 32; ++e) top = fmaxf(top, fabsf(s[e]));
+                        if (__all_sync(FULL, top <= cap.near_)) {
+#pragma unroll
+                            for (int e = c * 32; e < c * 32 + 32; e += 2) {
+                                const float2 y = score_capped_near(make_float2(s[e], s[e + 1]), cap);
+                                s[e] = y.x, s[e + 1] = y.y;
+                            }
+                        } else {
+#pragma unroll
+                            for (int e = c * 32; e < c * 32 + 32; ++e) s[e] = score_capped(s[e], cap);
+                        }
+                    }
                 }
                 const int key0 = j * FT_KEYS;
                 const bool masked = key0 + FT_KEYS - 1 > p0 || key0 + FT_KEYS - 1 > seq_hi ||

@@ -249,19 +249,49 @@ __device__ __forceinline__ float gate_mul_fast(float g, float u, const GateAct a
 }
 
 // Soft-capped attention scores, cap * tanh(s / cap), as the bfloat16 attention kernels apply them to their
-// float32 scores: `in` takes a product of query and key to s / cap, `out` is the cap in the softmax's units
-// (times log2 e).  tanh(x) = 1 - 2 / (1 + e^2x): absolute error of a few float32 roundings of 1, so a score is
-// right to about 1e-6 of the cap; e^2x overflowing to infinity gives 1, vanishing gives -1.
+// float32 scores; the result is in the softmax's units (times log2 e).  score_capped holds for every score:
+// tanh(x) = 1 - 2 / (1 + e^2x), an absolute error of a few float32 roundings of 1, so a score is right to about
+// 1e-6 of the cap; e^2x overflowing to infinity gives 1, vanishing gives -1.  It costs two special-function
+// operations.  score_capped_near holds for scores within the cap, |x| <= 1, and costs none: tanh(x) = x P(x^2)
+// with P the polynomial of degree 6 that is closest to tanh(sqrt u) / sqrt u on [0, 1] (relative error 5e-8, by
+// the exchange algorithm), two scores at a time.
 struct ScoreCap {
-    float in, out;
+    float in, in2, out, near_;      // scale / cap, 2 log2 e scale / cap, log2 e cap, and the largest |q . k| that is near
 };
 static inline ScoreCap score_cap(float scale, float cap) {
-    ScoreCap c = {0.0f, 0.0f};
-    if (cap > 0.0f) c.in = scale / cap, c.out = cap * 1.4426950408889634f;
+    ScoreCap c = {0.0f, 0.0f, 0.0f, 0.0f};
+    if (cap > 0.0f) {
+        c.in = scale / cap, c.in2 = 2.0f * 1.4426950408889634f * c.in, c.out = cap * 1.4426950408889634f;
+        c.near_ = c.in > 0.0f ? 1.0f / c.in : 0.0f;
+    }
     return c;
 }
 __device__ __forceinline__ float score_capped(float qk, const ScoreCap c) {
-    return c.out * (1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * (c.in * qk))));
+    float e, r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(c.in2 * qk));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+    return fmaf(-2.0f * c.out, r, c.out);
+}
+// two float32 multiply-adds in one instruction
+__device__ __forceinline__ float2 fma_x2(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("{\n.reg .b64 a, b, c, d;\nmov.b64 a, {%2, %3};\nmov.b64 b, {%4, %5};\nmov.b64 c, {%6, %7};\n"
+        "fma.rn.f32x2 d, a, b, c;\nmov.b64 {%0, %1}, d;\n}"
+        : "=f"(d.x), "=f"(d.y)
+        : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+    return d;
+}
+__device__ __forceinline__ float2 score_capped_near(float2 qk, const ScoreCap c) {
+    const float2 zero = make_float2(0.0f, 0.0f);
+    auto both = [](float v) { return make_float2(v, v); };
+    const float2 x = fma_x2(qk, both(c.in), zero), u = fma_x2(x, x, zero);
+    float2 p = fma_x2(u, both(0.00104102258568f), both(-0.00620337898208f));
+    p = fma_x2(p, u, both(0.0202899803204f));
+    p = fma_x2(p, u, both(-0.053457029549f));
+    p = fma_x2(p, u, both(0.133252040772f));
+    p = fma_x2(p, u, both(-0.333328391536f));
+    p = fma_x2(p, u, both(0.999999950241f));
+    return fma_x2(fma_x2(p, x, zero), both(c.out), zero);
 }
 
 static inline int dtype_size(int dtype) { return dtype == BFI_F32 ? 4 : 2; }

@@ -5,8 +5,8 @@
 // sequence, thread (g, c) rows g, g + groups, ... of column c in shared memory.  The gates' logits come
 // as float32 rows [tokens][2 * heads] (input gates, then forget gates).
 //
-// bfi_mlstm_step is for steps in which every sequence brings one token: a block owns 32 columns and keeps
-// its part of the state in registers, asked for (with n, m and the gates' weight rows) before the wait
+// bfi_mlstm_step is for steps in which every sequence brings one token: a block owns 32 to 128 columns and
+// keeps its part of the state in registers, asked for (with n, m and the gates' weight rows) before the wait
 // for the kernel that makes q, k and v.  The gates' logits are made here, from the layer's input and the
 // head's two weight rows, so a step needs no product of its own for them.  Everything a token needs is
 // linear in the old state once the gates are known,
@@ -122,9 +122,30 @@ extern "C" int bfi_mlstm_scan(const void* proj, int dtype, long stride, int q_of
 // ------------------------------------------------------------------------------------------
 // One new token per sequence
 // ------------------------------------------------------------------------------------------
-#define MEM_STEP_COLS 32
-#define MEM_STEP_GROUPS 8
-#define MEM_STEP_THREADS (MEM_STEP_COLS * MEM_STEP_GROUPS)
+#define MEM_STEP_THREADS 256
+#define MEM_STEP_MAX_D 256
+
+// a row's part of the state: W neighbouring columns
+template <int W>
+struct MemCols {
+    float v[W];
+    __device__ __forceinline__ void zero() {
+#pragma unroll
+        for (int j = 0; j < W; ++j) v[j] = 0.0f;
+    }
+    __device__ __forceinline__ void load(const float* p) {
+        if (W == 4) {
+            const float4 x = *reinterpret_cast<const float4*>(p);
+            v[0] = x.x, v[1 % W] = x.y, v[2 % W] = x.z, v[3 % W] = x.w;
+        } else {
+            v[0] = *p;
+        }
+    }
+    __device__ __forceinline__ void store(float* p) const {
+        if (W == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1 % W], v[2 % W], v[3 % W]);
+        else *p = v[0];
+    }
+};
 
 // 8 consecutive values of either storage type, as they are in memory
 template <typename T>
@@ -159,32 +180,35 @@ struct MemRaw8<float> {
     }
 };
 
-// VEC: the input's and the weights' rows are cut into whole 16-byte pieces
-template <typename T, int RPT, bool VEC>
-__global__ void __launch_bounds__(MEM_STEP_THREADS)
+// A block owns CT * VW columns; thread (g, c) rows g, g + G, ... of columns c * VW .. + VW - 1.
+// VEC: the input's and the weights' rows are cut into whole 16-byte pieces.
+template <typename T, int VW, int CT, int RPT, bool VEC>
+__global__ void __launch_bounds__(MEM_STEP_THREADS, 2)
 mlstm_step_kernel(const T* __restrict__ proj, long stride, int q_off, int k_off, int v_off, const T* __restrict__ x, long x_stride,
                   const T* __restrict__ w_gate, int width, const MemGates gp, float q_scale, float* __restrict__ out, long out_stride,
                   float* __restrict__ state, float* __restrict__ tails, const int* __restrict__ cu_seqlens,
                   const int* __restrict__ seq_slot, int H, int D, int V, int v_blocks) {
     pdl_trigger();
-    __shared__ float qs[MEM_STEP_GROUPS * RPT], ks[MEM_STEP_GROUPS * RPT];
-    __shared__ float red[MEM_STEP_GROUPS][MEM_STEP_COLS];
-    __shared__ float sums[4][MEM_STEP_GROUPS];
+    constexpr int G = MEM_STEP_THREADS / CT, COLS = CT * VW, WARPS = MEM_STEP_THREADS / 32;
+    __shared__ float qs[G * RPT], ks[G * RPT];
+    __shared__ __align__(16) float red[WARPS][COLS];
+    __shared__ float sums[4][WARPS];
     __shared__ int last;
     const int seq = blockIdx.y;
     const int slot = seq_slot[seq];
     if (slot < 0) return;
     const int h = blockIdx.x / v_blocks;
-    const int v0 = (blockIdx.x - h * v_blocks) * MEM_STEP_COLS;
-    const int tid = threadIdx.x, c = tid & (MEM_STEP_COLS - 1), g = tid / MEM_STEP_COLS;
-    const bool col_ok = v0 + c < V;
-    float* sp = state + (((size_t)slot * H + h) * D) * V + v0 + c;
+    const int v0 = (blockIdx.x - h * v_blocks) * COLS;
+    const int tid = threadIdx.x, c = tid % CT, g = tid / CT, warp = tid >> 5, lane = tid & 31;
+    const bool col_ok = v0 + c * VW < V;
+    float* sp = state + (((size_t)slot * H + h) * D) * V + v0 + c * VW;
     float* tail = tails + ((size_t)slot * H + h) * (D + 2);
-    float S[RPT];
+    MemCols<VW> S[RPT];
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
-        const int d = g + MEM_STEP_GROUPS * i;
-        S[i] = (col_ok && d < D) ? sp[(size_t)d * V] : 0.0f;
+        const int d = g + G * i;
+        if (col_ok && d < D) S[i].load(sp + (size_t)d * V);
+        else S[i].zero();
     }
     const float n_old = tid < D ? tail[tid] : 0.0f;       // D <= 256: a row a thread
     const float m_old = tail[D];
@@ -206,7 +230,9 @@ mlstm_step_kernel(const T* __restrict__ proj, long stride, int q_off, int k_off,
         nq = n_old * qv;
         kq = kv * qv;
     }
-    const float vv = col_ok ? to_f32(row[v_off + (size_t)h * V + v0 + c]) : 0.0f;
+    float vv[VW];
+#pragma unroll
+    for (int j = 0; j < VW; ++j) vv[j] = col_ok ? to_f32(row[v_off + (size_t)h * V + v0 + c * VW + j]) : 0.0f;
     if (VEC) {
         MemRaw8<T> rx;
         if (tid * 8 < width) {
@@ -224,33 +250,49 @@ mlstm_step_kernel(const T* __restrict__ proj, long stride, int q_off, int k_off,
         }
     }
     zi = warp_sum(zi), zf = warp_sum(zf), nq = warp_sum(nq), kq = warp_sum(kq);
-    if (c == 0) sums[0][g] = zi, sums[1][g] = zf, sums[2][g] = nq, sums[3][g] = kq;
+    if (lane == 0) sums[0][warp] = zi, sums[1][warp] = zf, sums[2][warp] = nq, sums[3][warp] = kq;
     __syncthreads();
-    float acc = 0.0f;
+    float acc[VW];
+#pragma unroll
+    for (int j = 0; j < VW; ++j) acc[j] = 0.0f;
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
-        const int d = g + MEM_STEP_GROUPS * i;
-        if (d < D) acc = fmaf(S[i], qs[d], acc);
+        const int d = g + G * i;
+        const float qv = d < D ? qs[d] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < VW; ++j) acc[j] = fmaf(S[i].v[j], qv, acc[j]);
     }
-    red[g][c] = acc;
+#pragma unroll
+    for (int o = CT; o < 32; o <<= 1)                     // the warp's other rows of the same columns
+#pragma unroll
+        for (int j = 0; j < VW; ++j) acc[j] += __shfl_xor_sync(0xffffffffu, acc[j], o);
+    if (lane < CT)
+#pragma unroll
+        for (int j = 0; j < VW; ++j) red[warp][c * VW + j] = acc[j];
     zi = zf = nq = kq = 0.0f;
 #pragma unroll
-    for (int i = 0; i < MEM_STEP_GROUPS; ++i) zi += sums[0][i], zf += sums[1][i], nq += sums[2][i], kq += sums[3][i];
+    for (int i = 0; i < WARPS; ++i) zi += sums[0][i], zf += sums[1][i], nq += sums[2][i], kq += sums[3][i];
     const float gi = mem_log_input(gp, zi, h), gf = mem_log_forget(gp, zf, h);
     const float m = fmaxf(gf + m_old, gi);
     const float keep = expf(gf + m_old - m), put = expf(gi - m);
 #pragma unroll
     for (int i = 0; i < RPT; ++i) {
-        const int d = g + MEM_STEP_GROUPS * i;
-        if (d < D && col_ok) sp[(size_t)d * V] = fmaf(keep, S[i], put * ks[d] * vv);
+        const int d = g + G * i;
+        if (d < D && col_ok) {
+            const float kv = put * ks[d];
+#pragma unroll
+            for (int j = 0; j < VW; ++j) S[i].v[j] = fmaf(keep, S[i].v[j], kv * vv[j]);
+            S[i].store(sp + (size_t)d * V);
+        }
     }
     __syncthreads();
-    if (g == 0 && col_ok) {
+    if (tid < COLS && v0 + tid < V) {
         float o = 0.0f;
 #pragma unroll
-        for (int i = 0; i < MEM_STEP_GROUPS; ++i) o += red[i][c];
-        o = fmaf(keep, o, put * kq * vv);
-        out[(size_t)t * out_stride + (size_t)h * V + v0 + c] = o / mem_denominator(fmaf(keep, nq, put * kq), m);
+        for (int i = 0; i < WARPS; ++i) o += red[i][tid];
+        const float v = to_f32(row[v_off + (size_t)h * V + v0 + tid]);
+        o = fmaf(keep, o, put * kq * v);
+        out[(size_t)t * out_stride + (size_t)h * V + v0 + tid] = o / mem_denominator(fmaf(keep, nq, put * kq), m);
     }
     if (last) {
         if (tid < D) tail[tid] = fmaf(keep, n_old, put * ks[tid]);
@@ -262,16 +304,36 @@ template <typename T>
 static void launch_mem_step(const void* proj, long stride, int q_off, int k_off, int v_off, const void* x, long x_stride, const void* w_gate,
                             int width, const MemGates& gp, float q_scale, float* out, long out_stride, float* state, float* tails,
                             const int* cu_seqlens, const int* seq_slot, int n_seqs, int H, int D, int V, cudaStream_t stream) {
-    const int v_blocks = (V + MEM_STEP_COLS - 1) / MEM_STEP_COLS;
-    const dim3 grid(H * v_blocks, n_seqs), block(MEM_STEP_THREADS);
+    const dim3 block(MEM_STEP_THREADS);
     const bool vec = width % 8 == 0 && x_stride % 8 == 0 && ((uintptr_t)x & 15) == 0 && ((uintptr_t)w_gate & 15) == 0;
-#define BFI_MEM_STEP(R, VV)                                                                                                     \
-    bfi_launch(mlstm_step_kernel<T, R, VV>, grid, block, 0, stream, (const T*)proj, stride, q_off, k_off, v_off, (const T*)x, x_stride, \
-               (const T*)w_gate, width, gp, q_scale, out, out_stride, state, tails, cu_seqlens, seq_slot, H, D, V, v_blocks)
-#define BFI_MEM_STEP_R(R)          \
-    do {                           \
-        if (vec) BFI_MEM_STEP(R, true);  \
-        else BFI_MEM_STEP(R, false);     \
+#define BFI_MEM_STEP(VW, CT, R, VV)                                                                                             \
+    do {                                                                                                                        \
+        const int v_blocks = (V + VW * CT - 1) / (VW * CT);                                                                     \
+        bfi_launch(mlstm_step_kernel<T, VW, CT, R, VV>, dim3(H * v_blocks, n_seqs), block, 0, stream, (const T*)proj, stride, q_off, k_off, \
+                   v_off, (const T*)x, x_stride, (const T*)w_gate, width, gp, q_scale, out, out_stride, state, tails, cu_seqlens, seq_slot, \
+                   H, D, V, v_blocks);                                                                                          \
+    } while (0)
+    if (vec && V % 4 == 0 && ((uintptr_t)state & 15) == 0) {
+        // columns per block: as many as leave every SM a block (the gates are made once a block)
+        const long heads = (long)n_seqs * H, n_sm = bfi_sm_count();
+        if (V > 64 && D <= 128 && heads * ((V + 127) / 128) >= n_sm) {
+            if (D <= 64) BFI_MEM_STEP(4, 32, 8, true);
+            else BFI_MEM_STEP(4, 32, 16, true);
+        } else if (V > 32 && heads * ((V + 63) / 64) >= n_sm) {
+            if (D <= 64) BFI_MEM_STEP(4, 16, 4, true);
+            else if (D <= 128) BFI_MEM_STEP(4, 16, 8, true);
+            else BFI_MEM_STEP(4, 16, 16, true);
+        } else {
+            if (D <= 64) BFI_MEM_STEP(4, 8, 2, true);
+            else if (D <= 128) BFI_MEM_STEP(4, 8, 4, true);
+            else BFI_MEM_STEP(4, 8, 8, true);
+        }
+        return;
+    }
+#define BFI_MEM_STEP_R(R)                     \
+    do {                                      \
+        if (vec) BFI_MEM_STEP(1, 32, R, true); \
+        else BFI_MEM_STEP(1, 32, R, false);    \
     } while (0)
     if (D <= 32) BFI_MEM_STEP_R(4);
     else if (D <= 64) BFI_MEM_STEP_R(8);
@@ -292,7 +354,7 @@ extern "C" int bfi_mlstm_step(const void* proj, int dtype, long stride, int q_of
     BFI_REQUIRE(cap > 0.0f, "mlstm_step: the gates' cap must be positive");
     BFI_REQUIRE(out_stride >= (long)H * V && x_stride >= width, "mlstm_step: a row stride is shorter than the row");
     if (n_seqs <= 0) return 0;
-    if (D > MEM_STEP_GROUPS * 32 || n_seqs > 65535) return 2;
+    if (D > MEM_STEP_MAX_D || n_seqs > 65535) return 2;
     const MemGates gp = {bias_i, bias_f, cap};
     if (dtype == BFI_F32)
         launch_mem_step<float>(proj, stride, q_off, k_off, v_off, x, x_stride, w_gate, width, gp, q_scale, out, out_stride, state, tails,
