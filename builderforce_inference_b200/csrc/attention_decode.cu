@@ -234,7 +234,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
                 for (int c = 0; c < 2; ++c) {
                     const int key = key0 + j * 8 + 2 * t + c;
-                    float v = CAP ? score_capped(s[j][r * 2 + c], cap) : s[j][r * 2 + c] * scale_log2;
+                    float v = (CAP ? score_tanh(s[j][r * 2 + c], cap) : s[j][r * 2 + c]) * scale_log2;
                     if (!have_page || key > pos || (key < lo && key >= keep_first)) v = -INFINITY;
                     s[j][r * 2 + c] = v;
                     mx = fmaxf(mx, v);
@@ -417,7 +417,7 @@ static int launch_decode(const void* q, long q_stride, void* out, long out_strid
                                               cudaGetErrorString(e));
     }
     dim3 grid(max_splits, n_kv * head_chunks, n_seqs);
-    const float scale_log2 = scale * 1.4426950408889634f;
+    const float scale_log2 = score_scale(scale, softcap);
     const float sink_log2 = sink * 1.4426950408889634f;       // -inf: no sink
     bfi_launch(kernel, grid, dim3(AD_THREADS), need, stream, mk, mv, (const bf16*)q, q_stride, (bf16*)out, out_stride,
                block_table, table_stride, seq_slot, seq_start, n_q, n_kv, window, keep_first, scale_log2, sink_log2, head_chunks, part_o, part_ml,

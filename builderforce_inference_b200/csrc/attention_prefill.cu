@@ -160,7 +160,7 @@ attention_prefill_kernel(const bf16* __restrict__ q, long q_stride, bf16* __rest
                 for (int j = 0; j < 8; ++j)
 #pragma unroll
                     for (int c = 0; c < 2; ++c) {
-                        float v = CAP ? score_capped(s[j][r * 2 + c], cap) : s[j][r * 2 + c] * scale_log2;
+                        float v = (CAP ? score_tanh(s[j][r * 2 + c], cap) : s[j][r * 2 + c]) * scale_log2;
                         if (need_mask) {
                             const int key = key_lo + j * 8 + 2 * t + c;
                             if (key > pos_r[r] || (key < lo_r[r] && key >= keep_first)) v = -INFINITY;
@@ -259,7 +259,7 @@ static int launch_prefill(const void* q, long q_stride, void* out, long out_stri
     dim3 grid((max_tokens + AP_QROWS - 1) / AP_QROWS, n_q, n_seqs);
     bfi_launch(kernel, grid, dim3(AD_THREADS), smem, stream, (const bf16*)q, q_stride, (bf16*)out, out_stride,
                (const bf16*)k_pages, (const bf16*)v_pages, block_table, table_stride, cu_seqlens, seq_slot, seq_start, n_q,
-               n_kv, window, keep_first, chunk, scale * 1.4426950408889634f, sink * 1.4426950408889634f, sinks, split_p,
+               n_kv, window, keep_first, chunk, score_scale(scale, softcap), sink * 1.4426950408889634f, sinks, split_p,
                score_cap(scale, softcap));
     return bfi_check_launch("attention_prefill");
 }

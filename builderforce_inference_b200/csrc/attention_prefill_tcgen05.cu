@@ -69,6 +69,14 @@ __device__ __forceinline__ void tmem_st32(uint32_t taddr, const uint32_t* v) {
           "r"(v[27]), "r"(v[28]), "r"(v[29]), "r"(v[30]), "r"(v[31])
         : "memory");
 }
+__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t* v) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
+        "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
+        ::"r"(taddr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]),
+          "r"(v[9]), "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15])
+        : "memory");
+}
 __device__ __forceinline__ void tmem_wait_ld() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
 __device__ __forceinline__ void tmem_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
@@ -175,7 +183,10 @@ struct FtItem {
 };
 
 // KEEP: there may be kept first positions (without them the kernel is the one for plain windows).
-// CAP: the scores are soft-capped as they are read; they are then in the exponent's units (scale_log2 is 1).
+// CAP: the scores become tanh(score / cap), and scale_log2 is the cap's.  The row's maximum is taken from the
+// scores as they are (the cap keeps their order); the second reading caps them, 32 keys at a time in a rolled
+// loop (ROLLED), since the unrolled form's instructions no longer come from the cache, and leaves P where the
+// scores of the same 32 keys were.
 template <int D, bool SPLIT_P, bool KEEP, bool CAP>
 __global__ void __launch_bounds__(FT_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
@@ -188,6 +199,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     constexpr int BOXES = D / 64;
     constexpr int TILE_BYTES = BOXES * FT_BOX_BYTES;       // a Q tile, a K tile or a V tile
     constexpr int PAGE_BYTES = FT_PAGE * 128;              // one page's rows inside a box
+    constexpr bool ROLLED = CAP;
     constexpr int S_COLS = FT_KEYS;                        // columns of one S buffer
     constexpr int O_COL = 2 * S_COLS;                      // the two O buffers behind the two S buffers
     constexpr uint32_t FULL = 0xffffffffu;
@@ -482,11 +494,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     const uint32_t p_addr = tmem_base + b * S_COLS;
 #pragma unroll
                     for (int kk = 0; kk < FT_KEYS / 16; ++kk)       // 16 keys per step: 8 columns of packed P, 2048 bytes of V
-                        umma_bf16_a_tmem(o_addr, p_addr + kk * 8, vd + (uint64_t)(kk * 2048 >> 4), idesc_o, (i > 0 || kk > 0));
+                        umma_bf16_a_tmem(o_addr, p_addr + (ROLLED ? (kk >> 1) * 32 + (kk & 1) * 8 : kk * 8), vd + (uint64_t)(kk * 2048 >> 4), idesc_o, (i > 0 || kk > 0));
                     if (SPLIT_P) {
 #pragma unroll
                         for (int kk = 0; kk < FT_KEYS / 16; ++kk)
-                            umma_bf16_a_tmem(o_addr, p_addr + FT_KEYS / 2 + kk * 8, vd + (uint64_t)(kk * 2048 >> 4), idesc_o, 1u);
+                            umma_bf16_a_tmem(o_addr, p_addr + (ROLLED ? (kk >> 1) * 32 + (kk & 1) * 8 + 16 : FT_KEYS / 2 + kk * 8),
+                                             vd + (uint64_t)(kk * 2048 >> 4), idesc_o, 1u);
                     }
                     umma_commit(&v_empty[b]);
                     umma_commit(o_tile);
@@ -541,24 +554,6 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
                 for (int c = 0; c < FT_KEYS / 32; ++c) tmem_ld32(s_addr + c * 32, s + c * 32);
                 tmem_wait_ld();
-                if (CAP) {
-#pragma unroll
-                    for (int c = 0; c < FT_KEYS / 32; ++c) {          // 32 keys at a time: scores near zero need no special functions
-                        float top = 0.0f;
-#pragma unroll
-                        for (int e = c * 32; e < c * 32 + 32; ++e) top = fmaxf(top, fabsf(s[e]));
-                        if (__all_sync(FULL, top <= cap.near_)) {
-#pragma unroll
-                            for (int e = c * 32; e < c * 32 + 32; e += 2) {
-                                const float2 y = score_capped_near(make_float2(s[e], s[e + 1]), cap);
-                                s[e] = y.x, s[e + 1] = y.y;
-                            }
-                        } else {
-#pragma unroll
-                            for (int e = c * 32; e < c * 32 + 32; ++e) s[e] = score_capped(s[e], cap);
-                        }
-                    }
-                }
                 const int key0 = j * FT_KEYS;
                 const bool masked = key0 + FT_KEYS - 1 > p0 || key0 + FT_KEYS - 1 > seq_hi ||
                                     (window > 0 && key0 < p0 + FT_ROWS - 1 - window + 1);
@@ -576,6 +571,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 float mx = s[0];
 #pragma unroll
                 for (int e = 1; e < FT_KEYS; ++e) mx = fmaxf(mx, s[e]);
+                if (CAP) mx = mx > -INFINITY ? score_tanh(mx, cap) : mx;       // the cap keeps the order
                 // raise the running maximum only when a score would otherwise exceed 2^8 after the shift
                 const bool raise = mx > -INFINITY && (m_used == -INFINITY || (mx - m_used) * scale_log2 > FT_RESCALE_ABOVE);
                 if (__any_sync(FULL, raise && i > 0)) {
@@ -604,7 +600,45 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 }
                 const float mc = m_used == -INFINITY ? 0.0f : m_used * scale_log2;
                 float sum = 0.0f;
-                if (SPLIT_P) {
+                if (ROLLED) {
+                    const int hi = pos_r - key0, lo = lo_r - key0, keep = keep_first - key0;
+#pragma unroll 1
+                    for (int c = 0; c < FT_KEYS / 32; ++c) {
+                        float x[32];
+                        uint32_t pk[32];
+                        tmem_ld32(s_addr + c * 32, x);
+                        tmem_wait_ld();
+                        if (CAP) {
+                            float top[4] = {};
+#pragma unroll
+                            for (int e = 0; e < 32; ++e) top[e & 3] = fmaxf(top[e & 3], fabsf(x[e]));
+                            if (__all_sync(FULL, fmaxf(fmaxf(top[0], top[1]), fmaxf(top[2], top[3])) <= cap.near_)) {
+#pragma unroll
+                                for (int e = 0; e < 32; e += 4) score_tanh_near(x + e, cap);
+                            } else {
+#pragma unroll
+                                for (int e = 0; e < 32; ++e) x[e] = score_tanh(x[e], cap);
+                            }
+                        }
+                        if (masked && !__all_sync(FULL, c * 32 + 31 <= hi && (c * 32 >= lo || (KEEP && c * 32 + 31 < keep)))) {
+#pragma unroll
+                            for (int e = 0; e < 32; ++e) {
+                                const int k = c * 32 + e;
+                                x[e] = (k > hi || (k < lo && (!KEEP || k >= keep))) ? -INFINITY : x[e];
+                            }
+                        }
+#pragma unroll
+                        for (int e = 0; e < 32; e += 2) {
+                            const float a = ft_exp2(fmaf(x[e], scale_log2, -mc)), c2 = ft_exp2(fmaf(x[e + 1], scale_log2, -mc));
+                            sum += a + c2;
+                            const uint32_t p2 = ft_pack(a, c2);
+                            pk[e >> 1] = p2;
+                            if (SPLIT_P) pk[16 + (e >> 1)] = ft_pack(a - __uint_as_float(p2 << 16), c2 - __uint_as_float(p2 & 0xffff0000u));
+                        }
+                        if (SPLIT_P) tmem_st32(s_addr + c * 32, pk);
+                        else tmem_st16(s_addr + c * 32, pk);
+                    }
+                } else if (SPLIT_P) {
                     // 64 keys at a time, so that the two terms fit beside the scores still to come
 #pragma unroll
                     for (int c = 0; c < FT_KEYS / 64; ++c) {
@@ -716,7 +750,7 @@ static int launch_prefill_tc(const void* qkv, long q_stride, void* out, long out
     dim3 grid((unsigned)(items < n_sm ? items : n_sm));      // one block per SM, each drawing items until none is left
     bfi_launch(kernel, grid, dim3(FT_THREADS), smem, stream, mq, mk, mv, (bf16*)out, out_stride, block_table, table_stride,
                cu_seqlens, seq_slot, seq_start, n_seqs, max_tiles, n_q, n_kv, window, keep_first,
-               CAP ? 1.0f : scale * 1.4426950408889634f, sink * 1.4426950408889634f, (uint32_t)lbo, (uint32_t)sbo, status, status + 1, waits,
+               score_scale(scale, softcap), sink * 1.4426950408889634f, (uint32_t)lbo, (uint32_t)sbo, status, status + 1, waits,
                score_cap(scale, softcap));
     return bfi_check_launch("attention_prefill_tcgen05");
 }

@@ -249,49 +249,45 @@ __device__ __forceinline__ float gate_mul_fast(float g, float u, const GateAct a
 }
 
 // Soft-capped attention scores, cap * tanh(s / cap), as the bfloat16 attention kernels apply them to their
-// float32 scores; the result is in the softmax's units (times log2 e).  score_capped holds for every score:
-// tanh(x) = 1 - 2 / (1 + e^2x), an absolute error of a few float32 roundings of 1, so a score is right to about
-// 1e-6 of the cap; e^2x overflowing to infinity gives 1, vanishing gives -1.  It costs two special-function
-// operations.  score_capped_near holds for scores within the cap, |x| <= 1, and costs none: tanh(x) = x P(x^2)
-// with P the polynomial of degree 6 that is closest to tanh(sqrt u) / sqrt u on [0, 1] (relative error 5e-8, by
-// the exchange algorithm), two scores at a time.
+// float32 scores: these give the tanh, and the softmax's scale is then the cap (score_scale).  score_tanh holds
+// for every score: tanh(x) = 1 - 2 / (1 + e^2x), an absolute error of a few float32 roundings of 1, so a score is
+// right to about 1e-6 of the cap; e^2x overflowing to infinity gives 1, vanishing gives -1.  It costs two
+// special-function operations.  score_tanh_near holds for scores within the cap, |x| <= 1, and costs none:
+// tanh(x) = x P(x^2) with P the polynomial of degree 6 that is closest to tanh(sqrt u) / sqrt u on [0, 1]
+// (relative error 5e-8, by the exchange algorithm).
 struct ScoreCap {
-    float in, in2, out, near_;      // scale / cap, 2 log2 e scale / cap, log2 e cap, and the largest |q . k| that is near
+    float in, in2, near_;      // scale / cap, 2 log2 e scale / cap, and the largest |q . k| that is near
 };
 static inline ScoreCap score_cap(float scale, float cap) {
-    ScoreCap c = {0.0f, 0.0f, 0.0f, 0.0f};
-    if (cap > 0.0f) {
-        c.in = scale / cap, c.in2 = 2.0f * 1.4426950408889634f * c.in, c.out = cap * 1.4426950408889634f;
-        c.near_ = c.in > 0.0f ? 1.0f / c.in : 0.0f;
-    }
+    ScoreCap c = {0.0f, 0.0f, 0.0f};
+    if (cap > 0.0f) c.in = scale / cap, c.in2 = 2.0f * 1.4426950408889634f * c.in, c.near_ = c.in > 0.0f ? 1.0f / c.in : 0.0f;
     return c;
 }
-__device__ __forceinline__ float score_capped(float qk, const ScoreCap c) {
+// what the softmax multiplies q . k (or its tanh) by, in units of log2 e
+static inline float score_scale(float scale, float cap) { return (cap > 0.0f ? cap : scale) * 1.4426950408889634f; }
+__device__ __forceinline__ float score_tanh(float qk, const ScoreCap c) {
     float e, r;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(c.in2 * qk));
     asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
-    return fmaf(-2.0f * c.out, r, c.out);
+    return fmaf(-2.0f, r, 1.0f);
 }
-// two float32 multiply-adds in one instruction
-__device__ __forceinline__ float2 fma_x2(float2 a, float2 b, float2 c) {
-    float2 d;
-    asm("{\n.reg .b64 a, b, c, d;\nmov.b64 a, {%2, %3};\nmov.b64 b, {%4, %5};\nmov.b64 c, {%6, %7};\n"
-        "fma.rn.f32x2 d, a, b, c;\nmov.b64 {%0, %1}, d;\n}"
-        : "=f"(d.x), "=f"(d.y)
-        : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
-    return d;
-}
-__device__ __forceinline__ float2 score_capped_near(float2 qk, const ScoreCap c) {
-    const float2 zero = make_float2(0.0f, 0.0f);
-    auto both = [](float v) { return make_float2(v, v); };
-    const float2 x = fma_x2(qk, both(c.in), zero), u = fma_x2(x, x, zero);
-    float2 p = fma_x2(u, both(0.00104102258568f), both(-0.00620337898208f));
-    p = fma_x2(p, u, both(0.0202899803204f));
-    p = fma_x2(p, u, both(-0.053457029549f));
-    p = fma_x2(p, u, both(0.133252040772f));
-    p = fma_x2(p, u, both(-0.333328391536f));
-    p = fma_x2(p, u, both(0.999999950241f));
-    return fma_x2(fma_x2(p, x, zero), both(c.out), zero);
+// Four scores in place, step by step side by side: written out, so that no step waits for the one before it.
+__device__ __forceinline__ void score_tanh_near(float* qk, const ScoreCap c) {
+#define BFI_TANH_STEP(COEF)               \
+    "fma.rn.f32 p0, p0, u0, " COEF ";\n"  \
+    "fma.rn.f32 p1, p1, u1, " COEF ";\n"  \
+    "fma.rn.f32 p2, p2, u2, " COEF ";\n"  \
+    "fma.rn.f32 p3, p3, u3, " COEF ";\n"
+    // coefficients from u^6 down: 1.0410226e-3, -6.2033790e-3, 2.0289980e-2, -5.3457030e-2, 0.13325204, -0.33332839, 0.99999995
+    asm volatile("{\n.reg .f32 u0, u1, u2, u3, p0, p1, p2, p3;\n"
+        "mul.rn.f32 %0, %0, %4;\nmul.rn.f32 %1, %1, %4;\nmul.rn.f32 %2, %2, %4;\nmul.rn.f32 %3, %3, %4;\n"
+        "mul.rn.f32 u0, %0, %0;\nmul.rn.f32 u1, %1, %1;\nmul.rn.f32 u2, %2, %2;\nmul.rn.f32 u3, %3, %3;\n"
+        "fma.rn.f32 p0, u0, 0f3A8872EC, 0fBBCB45B7;\nfma.rn.f32 p1, u1, 0f3A8872EC, 0fBBCB45B7;\nfma.rn.f32 p2, u2, 0f3A8872EC, 0fBBCB45B7;\nfma.rn.f32 p3, u3, 0f3A8872EC, 0fBBCB45B7;\n"
+        BFI_TANH_STEP("0f3CA6372C") BFI_TANH_STEP("0fBD5AF5C3") BFI_TANH_STEP("0f3E087339") BFI_TANH_STEP("0fBEAAAA05") BFI_TANH_STEP("0f3F7FFFFF")
+        "mul.rn.f32 %0, %0, p0;\nmul.rn.f32 %1, %1, p1;\nmul.rn.f32 %2, %2, p2;\nmul.rn.f32 %3, %3, p3;\n}"
+        : "+f"(qk[0]), "+f"(qk[1]), "+f"(qk[2]), "+f"(qk[3])
+        : "f"(c.in));
+#undef BFI_TANH_STEP
 }
 
 static inline int dtype_size(int dtype) { return dtype == BFI_F32 ? 4 : 2; }
