@@ -185,8 +185,7 @@ struct FtItem {
 // KEEP: there may be kept first positions (without them the kernel is the one for plain windows).
 // CAP: the scores become tanh(score / cap), and scale_log2 is the cap's.  The row's maximum is taken from the
 // scores as they are (the cap keeps their order); the second reading caps them, 32 keys at a time in a rolled
-// loop (ROLLED), since the unrolled form's instructions no longer come from the cache, and leaves P where the
-// scores of the same 32 keys were.
+// loop (ROLLED; unrolled it took a third longer), and leaves P where the scores of the same 32 keys were.
 template <int D, bool SPLIT_P, bool KEEP, bool CAP>
 __global__ void __launch_bounds__(FT_THREADS, 1)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
